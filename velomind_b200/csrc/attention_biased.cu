@@ -4,6 +4,7 @@
 //   q_h <- q_h / rms(q_h) * wq,  k_g <- k_g / rms(k_g) * wk          per head, one weight vector for all heads
 //   v   <- (1 - lambda) v + lambda v_first                            optional: the values of an earlier layer blended in
 //   score(i, j) = scale q_i . k_j + rel[bucket(i - j), h]             bucket: a table from the distance to a row of `rel`
+//                                 - slope[h] (i - j)                  optional: a bias linear in the distance, one slope per head
 //   i sees j  iff  j <= i and (i - j < window  or  j < keep_first)    window 0: every earlier key
 //   out_i = softmax_j(score) v_j
 //
@@ -78,7 +79,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
                                    const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                                    const int* __restrict__ seq_of_token, const float* __restrict__ rel, const int* __restrict__ bucket_of, int far,
                                    T* __restrict__ out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
-                                   int n_pages, const float* __restrict__ sink, int v_stride, int* __restrict__ err) {
+                                   int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes, int v_stride, int* __restrict__ err) {
     extern __shared__ float qs_all[];                       // ATT_WARPS x Dk
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long w = (long long)blockIdx.x * ATT_WARPS + warp;
@@ -94,6 +95,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
     const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;      // the window is [lo, pos]
     const int kept = min(keep_first, lo);                                             // keys [0, kept) are seen although outside it
     const int first_window_chunk = (lo / 32) * 32;
+    const float slope = slopes ? slopes[h] : 0.f;
     float m = -INFINITY, l = 0.f;
     float acc[EPL];
 #pragma unroll
@@ -116,6 +118,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
             float a = 0.f;
             for (int d = 0; d < Dk; ++d) a = fmaf(qs[d], vm_to_float(krow[d]), a);
             if (rel) a += rel[(size_t)bucket_of[min(pos - j, far)] * H + h];
+            if (slopes) a = fmaf(-slope, (float)(pos - j), a);
             s = a;
         }
         const float m_new = fmaxf(m, vm_warp_max(s));
@@ -156,7 +159,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
 template <typename T>
 int launch_biased(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                   const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, void* out, int n_tokens, int H,
-                  int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, const float* sink, int v_stride, int* err,
+                  int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, const float* sink, const float* slopes, int v_stride, int* err,
                   cudaStream_t stream) {
     const long long warps = (long long)n_tokens * H;
     const int blocks = (int)((warps + ATT_WARPS - 1) / ATT_WARPS);
@@ -168,7 +171,7 @@ int launch_biased(const void* q, int q_row_stride, const void* kpages, const voi
         attn_biased_kernel<T, E><<<blocks, ATT_WARPS * 32, smem, stream>>>((const T*)q, q_row_stride, (const T*)kpages, (const T*)vpages, \
                                                                            block_table, max_blocks, positions, seq_of_token, rel,       \
                                                                            bucket_of, far, (T*)out, n_tokens, H, Hkv, Dk, Dv, scale,     \
-                                                                           window, keep_first, n_pages, sink, v_stride, err);            \
+                                                                           window, keep_first, n_pages, sink, slopes, v_stride, err);    \
         break;
     switch (epl) {
         VM_ATT_CASE(1) VM_ATT_CASE(2) VM_ATT_CASE(3) VM_ATT_CASE(4) VM_ATT_CASE(5) VM_ATT_CASE(6) VM_ATT_CASE(7) VM_ATT_CASE(8)
@@ -208,16 +211,17 @@ VM_API int vm_attention_biased_generic(const void* q, int q_row_stride, const vo
                                        const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, void* out,
                                        int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages,
                                        int act_dtype, int* err, cudaStream_t stream) {
-    return vm_attention_sink_generic(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, nullptr, 0, out,
+    return vm_attention_sink_generic(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, nullptr, nullptr, 0, out,
                                      n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, act_dtype, err, stream);
 }
 
 // The same with a sink and values that may lie inside the key rows.  sink float32 [H] (null: none): exp(sink[h]) is one more term
 // of head h's softmax denominator, without a key or a value, not scaled.  v_row_stride: elements from one token's value row to the
 // next in `vpages` (0: Dv); with vpages == kpages and v_row_stride == Dk a token's value is the first Dv values of its key row.
+// slopes float32 [H] (null: none): slopes[h] * (i - j) is taken off head h's score of key j.
 VM_API int vm_attention_sink_generic(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                                      const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, const float* sink,
-                                     int v_row_stride, void* out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
+                                     const float* slopes, int v_row_stride, void* out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
                                      int n_pages, int act_dtype, int* err, cudaStream_t stream) {
     const int v_stride = v_row_stride > 0 ? v_row_stride : Dv;
     if (v_stride < Dv) return VM_ERR_BAD_ARG;
@@ -226,9 +230,9 @@ VM_API int vm_attention_sink_generic(const void* q, int q_row_stride, const void
     if ((rel != nullptr) != (bucket_of != nullptr) || (rel && far < 0)) return VM_ERR_BAD_ARG;
     if (act_dtype == VM_F32)
         return launch_biased<float>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, out, n_tokens, H,
-                                    Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, v_stride, err, stream);
+                                    Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err, stream);
     if (act_dtype == VM_BF16)
         return launch_biased<__nv_bfloat16>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, out,
-                                            n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, v_stride, err, stream);
+                                            n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err, stream);
     return VM_ERR_UNSUPPORTED;
 }

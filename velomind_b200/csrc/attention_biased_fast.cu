@@ -1,6 +1,8 @@
 // The bfloat16 kernels of the windowed attention with a distance bias and kept first tokens (arithmetic and arguments as in
 // attention_biased.cu): prompts on the tensor cores, decode steps with the keys of one query dealt out to the warps of a CTA.
 //
+// Both take, beside or instead of the table, a bias linear in the distance: slope[h] (i - j) comes off head h's score.
+//
 // Prompts.  One CTA owns 64 consecutive new tokens of one sequence and one query head; its four warps own 16 query rows
 // each.  The key blocks a tile can see are the pages of the kept first tokens and the pages its rows' windows touch; they
 // arrive one cache page (64 tokens of one kv head) at a time through cp.async into double-buffered shared memory, keys with
@@ -39,7 +41,8 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
                            const __nv_bfloat16* __restrict__ vpages, const int* __restrict__ block_table, int max_blocks,
                            const int* __restrict__ positions, const int* __restrict__ cu_tokens, int B, const float* __restrict__ rel,
                            const int* __restrict__ bucket_of, int far, int rel_rows, __nv_bfloat16* __restrict__ out, int H, int Hkv,
-                           float scale_log2, int window, int keep_first, int n_pages, const float* __restrict__ sink, int* __restrict__ err) {
+                           float scale_log2, int window, int keep_first, int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes,
+                           int* __restrict__ err) {
     constexpr int KP = DK + 8, VP = VK ? KP : DV + 8;     // padded rows: an odd number of 16-byte units -> no ldmatrix conflicts
     constexpr int KCH = DK / 8, VCH = DV / 8;   // 16-byte chunks per row
     constexpr float LOG2E = 1.4426950408889634f;
@@ -49,7 +52,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
     __nv_bfloat16* sV = sK + 2 * BN * KP;                                // [2][BN][VP]
     float* sBias = reinterpret_cast<float*>(VK ? sV : sV + 2 * BN * VP);  // direct: [far + 1] by distance; else [rel_rows] by table row
     constexpr int THREADS = 128;
-    const bool biased = rel != nullptr;
+    const bool biased = rel != nullptr, sloped = slopes != nullptr;
     const bool direct = biased && far + 1 <= DIRECT_TABLE_MAX;
 
     // ---- which 64 tokens of which sequence (the last tiles of a sequence see the most keys: they are started first)
@@ -116,6 +119,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
     unsigned qa[DK / 16][4];
     bool q_loaded = false;
     const int warp_min_pos = pos0 + warp * 16, warp_max_pos = warp_min_pos + 15;
+    const float slope_log2 = sloped ? slopes[h] * LOG2E : 0.f;
 
     for (int step = 0; step < n_steps; ++step) {
         const int buf = step & 1;
@@ -163,6 +167,10 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
                         const int da = min(max(pos_a - key, 0), far), db = min(max(pos_b - key, 0), far);
                         ba = direct ? sBias[da] : sBias[bucket_of[da]];
                         bb = direct ? sBias[db] : sBias[bucket_of[db]];
+                    }
+                    if (sloped) {
+                        ba = fmaf(-slope_log2, (float)(pos_a - key), ba);
+                        bb = fmaf(-slope_log2, (float)(pos_b - key), bb);
                     }
                     s[nb][e] = see_a ? fmaf(s[nb][e], scale_log2, ba) : -INFINITY;
                     s[nb][2 + e] = see_b ? fmaf(s[nb][2 + e], scale_log2, bb) : -INFINITY;
@@ -232,8 +240,8 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
 template <int DK, int DV, bool VK>
 int launch_biased_prefill(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                           const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel, const int* bucket_of, int far,
-                          int rel_rows, void* out, int H, int Hkv, float scale, int window, int keep_first, int n_pages, const float* sink, int* err,
-                          cudaStream_t stream) {
+                          int rel_rows, void* out, int H, int Hkv, float scale, int window, int keep_first, int n_pages, const float* sink, const float* slopes,
+                          int* err, cudaStream_t stream) {
     const int table = rel ? (far + 1 <= DIRECT_TABLE_MAX ? far + 1 : rel_rows) : 0;
     const size_t smem = (size_t)(BM + 2 * BN) * (DK + 8) * sizeof(__nv_bfloat16) + (VK ? 0 : (size_t)2 * BN * (DV + 8) * sizeof(__nv_bfloat16)) +
                         (size_t)table * sizeof(float);
@@ -246,7 +254,8 @@ int launch_biased_prefill(const void* q, int q_row_stride, const void* kpages, c
     }
     attn_biased_prefill_kernel<DK, DV, VK><<<dim3(n_tiles, H), 128, smem, stream>>>(
         (const __nv_bfloat16*)q, q_row_stride, (const __nv_bfloat16*)kpages, (const __nv_bfloat16*)vpages, block_table, max_blocks, positions,
-        cu_tokens, B, rel, bucket_of, far, rel_rows, (__nv_bfloat16*)out, H, Hkv, scale * 1.4426950408889634f, window, keep_first, n_pages, sink, err);
+        cu_tokens, B, rel, bucket_of, far, rel_rows, (__nv_bfloat16*)out, H, Hkv, scale * 1.4426950408889634f, window, keep_first, n_pages, sink,
+        slopes, err);
     return vm_launch_status();
 }
 
@@ -260,7 +269,7 @@ attn_biased_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride,
                           const __nv_bfloat16* __restrict__ vpages, const int* __restrict__ block_table, int max_blocks,
                           const int* __restrict__ positions, const float* __restrict__ rel, const int* __restrict__ bucket_of, int far,
                           __nv_bfloat16* __restrict__ out, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages,
-                          const float* __restrict__ sink, int v_stride, int* __restrict__ err) {
+                          const float* __restrict__ sink, const float* __restrict__ slopes, int v_stride, int* __restrict__ err) {
     extern __shared__ __align__(16) float dsm[];            // [Dk] the query; then per warp: m, l, acc[Dv]
     float* qs = dsm;
     float* part = dsm + ((Dk + 3) & ~3);
@@ -283,6 +292,7 @@ attn_biased_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride,
 #pragma unroll
     for (int i = 0; i < VPL; ++i) acc[i][0] = acc[i][1] = 0.f;
     const bool vec = (Dk % 8) == 0, pairs = (Dv % 2) == 0;
+    const float slope = slopes ? slopes[h] : 0.f;
     for (int c = warp; c < n_chunks; c += DEC_WARPS) {
         const int base = (c < kept_chunks ? c : first_window_chunk + (c - kept_chunks)) * 32;
         const int blk = base / VM_PAGE_TOKENS;
@@ -314,6 +324,7 @@ attn_biased_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride,
                 for (int d = 0; d < Dk; ++d) a = fmaf(qs[d], __bfloat162float(krow[d]), a);
             }
             if (rel) a += rel[(size_t)bucket_of[min(pos - j, far)] * H + h];
+            if (slopes) a = fmaf(-slope, (float)(pos - j), a);
             s = a;
         }
         const float m_new = fmaxf(m, vm_warp_max(s));
@@ -406,14 +417,15 @@ VM_API int vm_attention_biased_prefill_bf16(const void* q, int q_row_stride, con
                                             const int* bucket_of, int far, int rel_rows, void* out, int H, int Hkv, int Dk, int Dv, float scale,
                                             int window, int keep_first, int n_pages, int* err, cudaStream_t stream) {
     return vm_attention_sink_prefill_bf16(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, cu_tokens, B, n_tiles, rel, bucket_of, far,
-                                          rel_rows, nullptr, 0, out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, err, stream);
+                                          rel_rows, nullptr, nullptr, 0, out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, err, stream);
 }
 
-// The same with a sink (float32 [H], null: none; exp(sink[h]) joins head h's denominator) and, with vpages == kpages and
+// The same with a sink (float32 [H], null: none; exp(sink[h]) joins head h's denominator), slopes (float32 [H], null: none; slopes[h] (i - j)
+// comes off the score) and, with vpages == kpages and
 // v_row_stride == Dk, values that are the first Dv values of the key rows (sizes: vm_attention_sink_prefill_fits).
 VM_API int vm_attention_sink_prefill_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table,
                                           int max_blocks, const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel,
-                                          const int* bucket_of, int far, int rel_rows, const float* sink, int v_row_stride, void* out, int H, int Hkv,
+                                          const int* bucket_of, int far, int rel_rows, const float* sink, const float* slopes, int v_row_stride, void* out, int H, int Hkv,
                                           int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err, cudaStream_t stream) {
     if (n_tiles <= 0 || B <= 0) return 0;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || (q_row_stride % 8) != 0 || window < 0 || keep_first < 0) return VM_ERR_UNSUPPORTED;
@@ -423,7 +435,7 @@ VM_API int vm_attention_sink_prefill_bf16(const void* q, int q_row_stride, const
 #define VM_BP(K, V, IN)                                                                                                                        \
     if (Dk == K && Dv == V && in_keys == IN)                                                                                                   \
         return launch_biased_prefill<K, V, IN>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, cu_tokens, B, n_tiles, rel, \
-                                               bucket_of, far, rel_rows, out, H, Hkv, scale, window, keep_first, n_pages, sink, err, stream);
+                                               bucket_of, far, rel_rows, out, H, Hkv, scale, window, keep_first, n_pages, sink, slopes, err, stream);
     VM_BP(32, 16, false) VM_BP(32, 32, false) VM_BP(32, 64, false) VM_BP(32, 128, false)
     VM_BP(64, 16, false) VM_BP(64, 32, false) VM_BP(64, 64, false) VM_BP(64, 128, false)
     VM_BP(96, 16, false) VM_BP(96, 32, false) VM_BP(96, 64, false) VM_BP(96, 128, false)
@@ -441,14 +453,14 @@ VM_API int vm_attention_biased_decode_bf16(const void* q, int q_row_stride, cons
                                            int max_blocks, const int* positions, const float* rel, const int* bucket_of, int far, void* out, int B,
                                            int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err,
                                            cudaStream_t stream) {
-    return vm_attention_sink_decode_bf16(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, rel, bucket_of, far, nullptr, 0, out, B, H, Hkv,
+    return vm_attention_sink_decode_bf16(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, rel, bucket_of, far, nullptr, nullptr, 0, out, B, H, Hkv,
                                          Dk, Dv, scale, window, keep_first, n_pages, err, stream);
 }
 
-// the same with a sink and a stride between value rows (0: Dv), as vm_attention_sink_generic
+// the same with a sink, slopes and a stride between value rows (0: Dv), as vm_attention_sink_generic
 VM_API int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table,
                                          int max_blocks, const int* positions, const float* rel, const int* bucket_of, int far, const float* sink,
-                                         int v_row_stride, void* out, int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
+                                         const float* slopes, int v_row_stride, void* out, int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
                                          int n_pages, int* err, cudaStream_t stream) {
     if (B <= 0) return 0;
     if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dk > 1024 || Dv <= 0 || Dv > 256 || window < 0 || keep_first < 0) return VM_ERR_UNSUPPORTED;
@@ -463,7 +475,7 @@ VM_API int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const 
     case V:                                                                                                                                   \
         e = vm_launch_pdl(attn_biased_decode_kernel<V>, grid, dim3(DEC_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, q_row_stride,      \
                           (const __nv_bfloat16*)kpages, (const __nv_bfloat16*)vpages, block_table, max_blocks, positions, rel, bucket_of, far, \
-                          (__nv_bfloat16*)out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, v_stride, err);                       \
+                          (__nv_bfloat16*)out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err);               \
         break;
     switch ((Dv + 63) / 64) {
         VM_BD(1) VM_BD(2) VM_BD(3) VM_BD(4)

@@ -305,3 +305,29 @@ VM_API int vm_convert(const void* in, int in_dtype, void* out, int out_dtype, lo
     else return VM_ERR_UNSUPPORTED;
     return vm_launch_status();
 }
+
+// ------------------------------------------------------------------------------------------------ soft cap
+// x <- cap tanh(x / cap), in place
+__global__ void soft_cap_kernel(float* __restrict__ x, long long n, float cap, int aligned) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const float inv = 1.0f / cap;
+    const long long n4 = aligned ? n >> 2 : 0;
+    float4* x4 = reinterpret_cast<float4*>(x);
+    const long long first = (long long)blockIdx.x * blockDim.x + threadIdx.x, step = (long long)gridDim.x * blockDim.x;
+    for (long long i = first; i < n4; i += step) {
+        float4 v = x4[i];
+        v.x = cap * tanhf(v.x * inv); v.y = cap * tanhf(v.y * inv); v.z = cap * tanhf(v.z * inv); v.w = cap * tanhf(v.w * inv);
+        x4[i] = v;
+    }
+    for (long long i = 4 * n4 + first; i < n; i += step) x[i] = cap * tanhf(x[i] * inv);
+}
+
+VM_API int vm_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (!(cap > 0.f)) return VM_ERR_BAD_ARG;
+    const long long want = (n / 4 + 255) / 256;
+    const int grid = (int)(want < 1 ? 1 : (want < 148 * 8 ? want : 148 * 8));
+    vm_launch_pdl(soft_cap_kernel, dim3(grid), dim3(256), 0, stream, x, n, cap, (uintptr_t)x % 16 == 0 ? 1 : 0);
+    return vm_launch_status();
+}

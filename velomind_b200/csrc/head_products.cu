@@ -3,7 +3,7 @@
 //     out[t, h, 0:N] = W_h x[t, h, 0:K]          W_h = w + h * w_head, stored [N, K] (rows along the sum) or [K, N]
 //
 // with what follows such a product in a latent-attention layer taken into the same launch:
-//   gate:  out[t, h, n] *= sigmoid(gate[t, h * N + n])                       (float32 gate rows)
+//   gate:  out[t, h, n] *= sigmoid(gate[t, h * N + n])                       (float32 gate rows; or gate[t, h], one number per head)
 //   tail:  out[t, h, N : N + tail] = x[t, h, K : K + tail], its first rotary_dim values turned by the token's position
 //          (the rotated part of a query that passes the key up-projection by)
 //
@@ -155,7 +155,7 @@ head_product_kn_pairs_kernel(const __nv_bfloat16* __restrict__ x, long long x_ld
 __global__ void __launch_bounds__(256)
 head_product_nk_kernel(const __nv_bfloat16* __restrict__ x, long long x_ld, int x_head, const __nv_bfloat16* __restrict__ w, long long w_head,
                        __nv_bfloat16* __restrict__ out, long long out_ld, int out_head, int T, int N, int K, const float* __restrict__ gate,
-                       long long gate_ld) {
+                       long long gate_ld, int gate_per_head) {
     extern __shared__ __align__(16) float xs[];          // [HP_TOKENS][K]
     const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockIdx.y * 8 + warp, t0 = blockIdx.z * HP_TOKENS;
     const __nv_bfloat16* row = w + (size_t)h * w_head + (size_t)min(n, N - 1) * K;
@@ -193,7 +193,7 @@ head_product_nk_kernel(const __nv_bfloat16* __restrict__ x, long long x_ld, int 
     }
     const int t = t0 + lane;
     if (lane < HP_TOKENS && t < T) {
-        if (gate) mine = mine / (1.0f + expf(-gate[(size_t)t * gate_ld + (size_t)h * N + n]));
+        if (gate) mine = mine / (1.0f + expf(-gate[(size_t)t * gate_ld + (gate_per_head ? (size_t)h : (size_t)h * N + n)]));
         out[(size_t)t * out_ld + (size_t)h * out_head + n] = __float2bfloat16_rn(mine);
     }
 }
@@ -201,10 +201,11 @@ head_product_nk_kernel(const __nv_bfloat16* __restrict__ x, long long x_ld, int 
 }  // namespace
 
 // x [T, x_ld] with head h's K (+ tail) values at h * x_head; out [T, out_ld] with head h's N (+ tail) values at h * out_head; both
-// bfloat16.  k_by_n: the heads' weights are stored [K, N] (else [N, K]); a gate goes with [N, K], a tail with [K, N].
+// bfloat16.  k_by_n: the heads' weights are stored [K, N] (else [N, K]); a gate (a number per value, or gate_per_head: per head) goes with
+// [N, K], a tail with [K, N].
 VM_API int vm_head_products_few(const void* x, long long x_ld, int x_head, const void* w, long long w_head, int k_by_n, void* out, long long out_ld,
-                                int out_head, int T, int N, int K, int H, const float* gate, long long gate_ld, int tail, const int* positions,
-                                const float* inv_freq, int rotary_dim, int pairing, cudaStream_t stream) {
+                                int out_head, int T, int N, int K, int H, const float* gate, long long gate_ld, int gate_per_head, int tail,
+                                const int* positions, const float* inv_freq, int rotary_dim, int pairing, cudaStream_t stream) {
     if (T <= 0 || H <= 0) return 0;
     if (N <= 0 || K <= 0 || tail < 0 || rotary_dim < 0 || rotary_dim % 2 || rotary_dim > tail || (rotary_dim > 0 && (!inv_freq || !positions)))
         return VM_ERR_BAD_ARG;
@@ -222,6 +223,6 @@ VM_API int vm_head_products_few(const void* x, long long x_ld, int x_head, const
                       (const __nv_bfloat16*)w, w_head, (__nv_bfloat16*)out, out_ld, out_head, T, N, K, tail, positions, inv_freq, rotary_dim, pairing);
     else
         vm_launch_pdl(head_product_nk_kernel, dim3(H, (N + 7) / 8, tiles), dim3(256), smem, stream, (const __nv_bfloat16*)x, x_ld, x_head,
-                      (const __nv_bfloat16*)w, w_head, (__nv_bfloat16*)out, out_ld, out_head, T, N, K, gate, gate_ld);
+                      (const __nv_bfloat16*)w, w_head, (__nv_bfloat16*)out, out_ld, out_head, T, N, K, gate, gate_ld, gate_per_head);
     return vm_launch_status();
 }

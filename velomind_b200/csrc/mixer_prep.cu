@@ -4,7 +4,7 @@
 //   row = [q | k | v] projected (float32), plus an optional bias per column
 //   row <- short causal convolution over time per channel (taps [C, K]; the K - 1 last projected rows of a sequence are kept)
 //   values that are the keys: v = k as it leaves the convolution
-//   q, k <- RMS norm over the WHOLE projection (all heads at once) with a weight per column
+//   q, k <- RMS norm over the WHOLE projection (all heads at once) with a weight per column; or every head divided by its root mean square
 //   q, k <- rotary positions on the first rotary_dim values of every head, either pairing, angles in float32
 //   q -> its own buffer (activation dtype); k, v -> the sequence's cache page
 //
@@ -21,7 +21,7 @@ __global__ void mixer_prepare_kernel(const float* __restrict__ proj, int ld, con
                                      const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ cu_tokens,
                                      const int* __restrict__ slots, const int* __restrict__ block_table, int max_blocks, T* __restrict__ q_out,
                                      T* __restrict__ kpages, T* __restrict__ vpages, int n_pages, int H, int G, int Dk, int Dv, int values_are_keys,
-                                     int keep_here, int* __restrict__ err) {
+                                     int unit_heads, int keep_here, int* __restrict__ err) {
     extern __shared__ float row[];           // C floats: q heads, k heads, v heads
     __shared__ float red[32];
     vm_pdl_launch_dependents();
@@ -91,6 +91,16 @@ __global__ void mixer_prepare_kernel(const float* __restrict__ proj, int ld, con
         __syncthreads();
         for (int c = threadIdx.x; c < nq + nk; c += blockDim.x) row[c] = c < nq ? row[c] * iq * q_norm[c] : row[c] * ik * k_norm[c - nq];
     }
+    if (unit_heads) {                                     // (a warp per head)
+        __syncthreads();
+        for (int head = threadIdx.x >> 5; head < H + G; head += blockDim.x >> 5) {
+            float* x = row + (size_t)head * Dk;
+            float ss = 0.f;
+            for (int i = threadIdx.x & 31; i < Dk; i += 32) ss += x[i] * x[i];
+            const float f = 1.0f / sqrtf(vm_warp_sum(ss) / (float)Dk + eps);
+            for (int i = threadIdx.x & 31; i < Dk; i += 32) x[i] *= f;
+        }
+    }
     __syncthreads();
     // 4. rotary positions on q and k heads, in place (a thread per pair)
     if (inv_freq && rotary_dim > 0) {
@@ -137,14 +147,16 @@ __global__ void mixer_keep_rows_kernel(const float* __restrict__ proj, int ld, i
 
 // proj float32 [T, ld]: columns [0, H Dk) queries, then G Dk keys, then (unless the values are the keys) G Dv values; bias float32 [C]
 // or null; taps float32 [C, K] or null (K taps; the K - 1 rows kept per sequence lie in state [slot, state_stride] at state_offset);
-// q_norm [H Dk], k_norm [G Dk] or both null; inv_freq [rotary_dim / 2] or null.  q_out [T, H Dk] and the pages in the activation dtype.
+// q_norm [H Dk], k_norm [G Dk] or both null; unit_heads: every q and k head divided by its root mean square.  G = 0: a row of queries alone
+// (the layer reads keys and values that another one wrote; no pages are given).  inv_freq [rotary_dim / 2] or null.  q_out [T, H Dk] and the pages in the activation dtype.
 VM_API int vm_mixer_prepare(const float* proj, int ld, const float* bias, const float* taps, int K, float* state, long long state_stride,
                             int state_offset, const float* q_norm, const float* k_norm, float eps, const float* inv_freq, int rotary_dim, int pairing,
                             const int* positions, const int* seq_of_token, const int* cu_tokens, const int* slots, const int* block_table,
                             int max_blocks, void* q_out, void* kpages, void* vpages, int n_pages, int T, int B, int H, int G, int Dk, int Dv,
-                            int values_are_keys, int one_token_each, int act_dtype, int* err, cudaStream_t stream) {
+                            int values_are_keys, int unit_heads, int one_token_each, int act_dtype, int* err, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (H <= 0 || G <= 0 || Dk <= 0 || Dv <= 0 || (values_are_keys && Dv != Dk)) return VM_ERR_BAD_ARG;
+    if (H <= 0 || G < 0 || Dk <= 0 || Dv <= 0 || (values_are_keys && Dv != Dk) || (G == 0 && (kpages || vpages))) return VM_ERR_BAD_ARG;
+    if (unit_heads && q_norm) return VM_ERR_BAD_ARG;
     if (taps && (K < 1 || K > PREP_MAX_TAPS || (K > 1 && !state))) return VM_ERR_BAD_ARG;
     if ((q_norm != nullptr) != (k_norm != nullptr)) return VM_ERR_BAD_ARG;
     if (inv_freq && (rotary_dim < 0 || rotary_dim > Dk || rotary_dim % 2)) return VM_ERR_BAD_ARG;
@@ -160,13 +172,13 @@ VM_API int vm_mixer_prepare(const float* proj, int ld, const float* bias, const 
         if (e != cudaSuccess) return (int)e;
         vm_launch_pdl(mixer_prepare_kernel<float>, dim3(T), dim3(threads), smem, stream, proj, ld, bias, taps, K, state, state_stride, state_offset, q_norm,
                       k_norm, eps, inv_freq, rotary_dim, pairing, positions, seq_of_token, cu_tokens, slots, block_table, max_blocks, (float*)q_out,
-                      (float*)kpages, (float*)vpages, n_pages, H, G, Dk, Dv, values_are_keys, keep_here, err);
+                      (float*)kpages, (float*)vpages, n_pages, H, G, Dk, Dv, values_are_keys, unit_heads, keep_here, err);
     } else if (act_dtype == VM_BF16) {
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(mixer_prepare_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         vm_launch_pdl(mixer_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, stream, proj, ld, bias, taps, K, state, state_stride, state_offset,
                       q_norm, k_norm, eps, inv_freq, rotary_dim, pairing, positions, seq_of_token, cu_tokens, slots, block_table, max_blocks,
-                      (__nv_bfloat16*)q_out, (__nv_bfloat16*)kpages, (__nv_bfloat16*)vpages, n_pages, H, G, Dk, Dv, values_are_keys, keep_here, err);
+                      (__nv_bfloat16*)q_out, (__nv_bfloat16*)kpages, (__nv_bfloat16*)vpages, n_pages, H, G, Dk, Dv, values_are_keys, unit_heads, keep_here, err);
     } else return VM_ERR_UNSUPPORTED;
     int st = vm_launch_status();
     if (st || K <= 1 || keep_here) return st;

@@ -4,6 +4,7 @@
 //       out_t = h_t + sum_j taps[:, j] * h_(t - K + 1 + j)        (zeros before the sequence's start)
 //     with the last K - 1 inputs of every sequence kept in a float32 state area from step to step;
 //   h += rmsnorm(y) * w, the residual sum of a normed sublayer output;
+//   the same sum followed by the next sublayer's norm, for layers with a norm on both sides of every sublayer;
 //   the polynomial activation  a N(z) + b N(z^2) + c N(z^3) + e, N = division of a token's row by its root mean square;
 //   rotation of a slice of every head's row (rotary positions on a part of the head), copied to another layout;
 //   multiplication by the sigmoid of a gate.
@@ -290,6 +291,123 @@ __global__ void norm_residual_conv_step_kernel(float* __restrict__ h, const Y* _
     out[(size_t)t * hid + c] = vm_from_float<T>(acc);
 }
 
+// ------------------------------------------------------------------------------------------------ h += rmsnorm(y + bias) * w_out;  out = rmsnorm(h) * w_in
+// A layer with a norm on both sides of its sublayers: the sum of one sublayer and the read of the next in one pass, one block per token.
+// bias float32 [hid] or null.  `rows` (null: all): block i makes row rows[i] of h and y into row i of out, and h stays as it is.
+__device__ __forceinline__ float4 ns_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ns_load4(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void ns_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void ns_store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<const unsigned*>(&a);
+    r.y = *reinterpret_cast<const unsigned*>(&b);
+    *reinterpret_cast<uint2*>(p) = r;
+}
+
+// rows of 4 n values: a thread keeps RUNS runs of four values of its row in registers (hid <= 4 * RUNS * blockDim)
+template <typename T, int RUNS>
+__global__ void __launch_bounds__(256)
+norm_sum_norm_vec_kernel(float* __restrict__ h, const T* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w_out, float eps_out,
+                         const float* __restrict__ w_in, float eps_in, T* __restrict__ out, const int* __restrict__ rows, int hid) {
+    __shared__ float red[32];
+    vm_pdl_launch_dependents();
+    float4 wo[RUNS], wi[RUNS], x[RUNS], s[RUNS];
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {                     // (weights are constants: they may be read before the wait)
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        wo[c] = wi[c] = x[c] = s[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i >= hid) continue;
+        wo[c] = ns_load4(w_out + i);
+        wi[c] = ns_load4(w_in + i);
+        if (bias) x[c] = ns_load4(bias + i);
+    }
+    vm_pdl_wait();
+    const size_t t = rows ? rows[blockIdx.x] : blockIdx.x;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        if (i >= hid) continue;
+        const float4 v = ns_load4(y + t * hid + i);
+        s[c] = ns_load4(h + t * hid + i);
+        x[c].x += v.x; x[c].y += v.y; x[c].z += v.z; x[c].w += v.w;
+        ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+    }
+    ss = vm_block_sum(ss, red);
+    const float fo = 1.0f / sqrtf(ss / (float)hid + eps_out);
+    float st = 0.f;
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        s[c].x += x[c].x * fo * wo[c].x; s[c].y += x[c].y * fo * wo[c].y; s[c].z += x[c].z * fo * wo[c].z; s[c].w += x[c].w * fo * wo[c].w;
+        if (i < hid && !rows) ns_store4(h + t * hid + i, s[c]);
+        st += s[c].x * s[c].x + s[c].y * s[c].y + s[c].z * s[c].z + s[c].w * s[c].w;
+    }
+    st = vm_block_sum(st, red);
+    const float fi = 1.0f / sqrtf(st / (float)hid + eps_in);
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        if (i >= hid) continue;
+        ns_store4(out + (size_t)blockIdx.x * hid + i, make_float4(s[c].x * fi * wi[c].x, s[c].y * fi * wi[c].y, s[c].z * fi * wi[c].z, s[c].w * fi * wi[c].w));
+    }
+}
+
+// any width; the row is walked three times (it comes out of L1 again)
+template <typename T>
+__global__ void norm_sum_norm_kernel(float* __restrict__ h, const T* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w_out,
+                                     float eps_out, const float* __restrict__ w_in, float eps_in, T* __restrict__ out, const int* __restrict__ rows, int hid) {
+    __shared__ float red[32];
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const size_t t = rows ? rows[blockIdx.x] : blockIdx.x;
+    const T* yr = y + t * hid;
+    float* hr = h + t * hid;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < hid; i += blockDim.x) {
+        const float v = vm_to_float(yr[i]) + (bias ? bias[i] : 0.f);
+        ss += v * v;
+    }
+    ss = vm_block_sum(ss, red);
+    const float fo = 1.0f / sqrtf(ss / (float)hid + eps_out);
+    float st = 0.f;
+    for (int i = threadIdx.x; i < hid; i += blockDim.x) {
+        const float v = hr[i] + (vm_to_float(yr[i]) + (bias ? bias[i] : 0.f)) * fo * w_out[i];
+        st += v * v;
+    }
+    st = vm_block_sum(st, red);
+    const float fi = 1.0f / sqrtf(st / (float)hid + eps_in);
+    for (int i = threadIdx.x; i < hid; i += blockDim.x) {
+        const float v = hr[i] + (vm_to_float(yr[i]) + (bias ? bias[i] : 0.f)) * fo * w_out[i];
+        if (!rows) hr[i] = v;
+        out[(size_t)blockIdx.x * hid + i] = vm_from_float<T>(v * fi * w_in[i]);
+    }
+}
+
+template <typename T>
+int launch_norm_sum_norm(float* h, const T* y, const float* bias, const float* w_out, float eps_out, const float* w_in, float eps_in, T* out, const int* rows,
+                         int n, int hid, cudaStream_t stream) {
+    const uintptr_t at = (uintptr_t)h | (uintptr_t)y | (uintptr_t)bias | (uintptr_t)w_out | (uintptr_t)w_in | (uintptr_t)out;
+    if (hid % 4 == 0 && at % 16 == 0 && hid <= 4096) {
+        const int threads = hid >= 1024 ? 256 : (hid >= 512 ? 128 : 64);
+        const int runs = (hid / 4 + threads - 1) / threads;
+#define VM_NSN(R_) \
+    vm_launch_pdl(norm_sum_norm_vec_kernel<T, R_>, dim3(n), dim3(threads), 0, stream, h, y, bias, w_out, eps_out, w_in, eps_in, out, rows, hid)
+        if (runs <= 1) VM_NSN(1);
+        else if (runs <= 2) VM_NSN(2);
+        else VM_NSN(4);
+#undef VM_NSN
+    } else {
+        vm_launch_pdl(norm_sum_norm_kernel<T>, dim3(n), dim3(hid >= 512 ? 256 : 128), 0, stream, h, y, bias, w_out, eps_out, w_in, eps_in, out, rows, hid);
+    }
+    return vm_launch_status();
+}
+
 // ------------------------------------------------------------------------------------------------ polynomial activation with unit-rms powers
 // one block per token; z [T, n] in Z (float32 or the activation dtype), out in T
 template <typename Z, typename T>
@@ -500,6 +618,18 @@ VM_API int vm_norm_residual_add(float* h, const void* y, long long ld, int y_dty
         vm_launch_pdl(norm_residual_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, stream, h, (const __nv_bfloat16*)y, ld, w, hid, eps);
     else return VM_ERR_UNSUPPORTED;
     return vm_launch_status();
+}
+
+// h float32 [T, hid] += rmsnorm(y + bias) * w_out; out [T, hid] = rmsnorm(h) * w_in.  y and out in act_dtype, bias float32 [hid] or null.
+// With `rows` (int32 [n]) only those n rows are made, into rows 0 .. n of out, and h is not written.
+VM_API int vm_norm_sum_norm(float* h, const void* y, const float* bias, const float* w_out, float eps_out, const float* w_in, float eps_in, void* out,
+                            const int* rows, int n, int hid, int act_dtype, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (hid <= 0 || !w_out || !w_in) return VM_ERR_BAD_ARG;
+    if (act_dtype == VM_F32) return launch_norm_sum_norm<float>(h, (const float*)y, bias, w_out, eps_out, w_in, eps_in, (float*)out, rows, n, hid, stream);
+    if (act_dtype == VM_BF16)
+        return launch_norm_sum_norm<__nv_bfloat16>(h, (const __nv_bfloat16*)y, bias, w_out, eps_out, w_in, eps_in, (__nv_bfloat16*)out, rows, n, hid, stream);
+    return VM_ERR_UNSUPPORTED;
 }
 
 // One token per sequence (token s is sequence s's): h += rmsnorm(y) * w, then out = h + conv(h) as vm_input_conv does for such a step,

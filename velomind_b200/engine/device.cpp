@@ -129,21 +129,32 @@ DeviceTensor BindContext::upload(const HostTensor& t, DType as) {
     return d;
 }
 
-DeviceTensor BindContext::upload_stacked(const std::vector<const HostTensor*>& parts, DType as) {
-    if (parts.size() == 1) return upload(*parts[0], as);
+DeviceTensor BindContext::upload_stacked(const std::vector<const HostTensor*>& parts, DType as, int row_multiple) {
+    if (parts.size() == 1 && row_multiple <= 1) return upload(*parts[0], as);
     long long rows = 0;
     const long long cols = parts[0]->shape.size() > 1 ? parts[0]->shape[1] : 1;
     for (const HostTensor* p : parts) rows += p->shape[0];
+    if (row_multiple > 1) rows = (rows + row_multiple - 1) / row_multiple * row_multiple;
     DeviceTensor d;
     d.dtype = as;
     d.shape = {rows, cols};
-    d.owner = std::make_shared<DeviceBuffer>(static_cast<size_t>(rows * cols) * dtype_size(as));
+    d.owner = std::make_shared<DeviceBuffer>(static_cast<size_t>(rows * cols) * dtype_size(as), /*zero=*/row_multiple > 1);
     d.ptr = d.owner->ptr;
     size_t off = 0;
     for (const HostTensor* p : parts) {
         copy_in(static_cast<char*>(d.ptr) + off, *p, as, stream);
         off += static_cast<size_t>(p->numel()) * dtype_size(as);
     }
+    return d;
+}
+
+DeviceTensor BindContext::upload_scaled(const HostTensor& t, float factor) {
+    const std::vector<uint8_t> bytes = converted(t, DType::F32);
+    std::vector<float> values(bytes.size() / sizeof(float));
+    std::memcpy(values.data(), bytes.data(), values.size() * sizeof(float));
+    for (float& v : values) v *= factor;
+    DeviceTensor d = upload_floats(values);
+    d.shape = t.shape;
     return d;
 }
 
@@ -508,7 +519,7 @@ void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const K
     if (ctx.act_dtype == DType::BF16 && ctx.one_token_each && Dk <= 1024 && Dv <= 256 && H <= 65535) {
         Timed t("attention_biased_decode_bf16", s);
         check(vm_attention_sink_decode_bf16(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, mask.rel, mask.bucket_of,
-                                            mask.far, mask.sink, mask.v_row_stride, out, ctx.B, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
+                                            mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.B, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
                                             kv.n_pages, ctx.err, s),
               "attention_biased_decode_bf16", s);
         return;
@@ -518,14 +529,14 @@ void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const K
         for (int b = 0; b < ctx.B; ++b) tiles += (ctx.host_cu_tokens[b + 1] - ctx.host_cu_tokens[b] + 63) / 64;
         Timed t("attention_biased_prefill_bf16", s);
         check(vm_attention_sink_prefill_bf16(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, ctx.cu_tokens, ctx.B,
-                                             static_cast<int>(tiles), mask.rel, mask.bucket_of, mask.far, mask.rows, mask.sink, mask.v_row_stride, out, H,
+                                             static_cast<int>(tiles), mask.rel, mask.bucket_of, mask.far, mask.rows, mask.sink, mask.slopes, mask.v_row_stride, out, H,
                                              Hkv, Dk, Dv, scale, mask.window, mask.keep_first, kv.n_pages, ctx.err, s),
               "attention_biased_prefill_bf16", s);
         return;
     }
     Timed t("attention_biased_generic", s);
     check(vm_attention_sink_generic(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, ctx.seq_of_token, mask.rel,
-                                    mask.bucket_of, mask.far, mask.sink, mask.v_row_stride, out, ctx.T, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
+                                    mask.bucket_of, mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.T, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
                                     kv.n_pages, code(ctx.act_dtype), ctx.err, s),
           "attention_biased_generic", s);
 }

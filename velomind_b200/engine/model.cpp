@@ -1,5 +1,6 @@
 // A decoder model built from a plan: embedding, layers run in the plan's order, final norm, head.
 // Nothing here names an architecture; the plan says which parts and which order.
+#include <algorithm>
 #include <cstdio>
 #include <cstdlib>
 
@@ -124,6 +125,23 @@ std::vector<CacheNeed> DecoderModel::cache_needs() const {
         need.state_floats += wiring;
         out.push_back(need);
     }
+    // a run that others read keeps what the farthest-looking of them needs
+    for (const ScheduleEntry& e : plan.schedule) {
+        if (e.cache_of < 0) continue;
+        CacheNeed& kept = out[e.cache_of];
+        const CacheNeed reader = layers[e.layer].parts.mixer->cache_need();
+        if (kept.kind == CacheNeed::None || reader.kind == CacheNeed::None) continue;
+        if (reader.kv_heads != kept.kv_heads || reader.key_dim != kept.key_dim || reader.value_dim != kept.value_dim)
+            throw ConfigError(format("a layer reads the keys and values of run %d, which have other sizes than its own", e.cache_of));
+        if (kept.kind == CacheNeed::All) continue;
+        if (reader.kind == CacheNeed::All) {
+            kept.kind = CacheNeed::All;
+            kept.window = kept.keep_first = 0;
+        } else {
+            kept.window = std::max(kept.window, reader.window);
+            kept.keep_first = std::max(kept.keep_first, reader.keep_first);
+        }
+    }
     if (embedding->state_floats() > 0) {             // what the embedding keeps per sequence: one more state area behind the runs'
         CacheNeed need;
         need.state_floats = embedding->state_floats();
@@ -189,6 +207,12 @@ void DecoderModel::forward(StepContext& ctx) {
                 pending = nullptr;
                 ctx.pending_mix = ctx.pending_out = nullptr;
             }
+            if (pending && ctx.pending_norm_weight) {
+                ops::norm_residual_add(h, pending, hid, ctx.act_dtype, ctx.pending_norm_weight, ctx.pending_norm_eps, ctx.T, static_cast<int>(hid), ctx.stream);
+                ctx.give(pending);
+                pending = nullptr;
+                ctx.pending_norm_weight = nullptr;
+            }
             dump_stream(ctx, h, pending != nullptr);
         }
     }
@@ -200,17 +224,24 @@ void DecoderModel::forward(StepContext& ctx) {
     }
     ctx.pending_mix = ctx.pending_out = nullptr;
     if (S > 1 && ctx.R > 0) ops::streams_sum_rows(h, ctx.stream_stride, S, ctx.logit_rows, ctx.R, static_cast<int>(hid), ctx.stream);   // copy 0 <- the sum, at the wanted rows
-    if (pending && ctx.pending_norm_weight) {        // the last layer's norm sits on its output: add its normed delta first
+    // the last layer's norm sits on its output: its normed delta joins the stream first (at the wanted rows alone, together with the final
+    // norm, where that is a root-mean-square norm: nothing reads the stream afterwards)
+    const float* final_weight = nullptr;
+    float final_eps = 0.f;
+    const bool joins = pending && ctx.pending_norm_weight && final_norm->as_rms(&final_weight, &final_eps);
+    if (pending && ctx.pending_norm_weight && !joins) {
         ops::norm_residual_add(h, pending, hid, ctx.act_dtype, ctx.pending_norm_weight, ctx.pending_norm_eps, ctx.T, static_cast<int>(hid), ctx.stream);
         ctx.give(pending);
         pending = nullptr;
     }
+    const float* last_weight = ctx.pending_norm_weight;
     ctx.pending_norm_weight = nullptr;
     // Final norm and head on the wanted rows (plus `pending`, a product not yet added to the residual stream).  A step that
     // wants no logits (a prompt cut into several steps) has a bucket of its own, so it asks for nothing here.
     if (ctx.R > 0) {
         void* rows = ctx.take(static_cast<long long>(ctx.R_cap) * hid, ctx.act_dtype);
-        final_norm->forward(ctx, h, pending, rows, ctx.logit_rows, ctx.R);
+        if (joins) ops::norm_sum_norm(h, pending, nullptr, last_weight, ctx.pending_norm_eps, final_weight, final_eps, rows, ctx.logit_rows, ctx.R, static_cast<int>(hid), ctx.act_dtype, ctx.stream);
+        else final_norm->forward(ctx, h, pending, rows, ctx.logit_rows, ctx.R);
         head->forward(ctx, rows, ctx.logits);
         ctx.give(rows);
     }

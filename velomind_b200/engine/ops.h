@@ -76,6 +76,14 @@ inline void norm_residual_add(float* h, const void* y, long long ld, DType y_dty
     check(vm_norm_residual_add(h, y, ld, code(y_dtype), w, T, hid, eps, s), "norm_residual_add", s);
 }
 
+// that sum followed by the next sublayer's norm: h += rmsnorm(y + bias) * w_out; out = rmsnorm(h) * w_in.  With `rows` only those n rows are
+// made, into the first n rows of out, and h stays as it is.
+inline void norm_sum_norm(float* h, const void* y, const float* bias, const float* w_out, float eps_out, const float* w_in, float eps_in, void* out,
+                          const int* rows, int n, int hid, DType act, cudaStream_t s) {
+    Timed t("norm_sum_norm", s);
+    check(vm_norm_sum_norm(h, y, bias, w_out, eps_out, w_in, eps_in, out, rows, n, hid, code(act), s), "norm_sum_norm", s);
+}
+
 // a step of one token per sequence: that sum and the next sublayer's input convolution in one launch
 inline void norm_residual_conv_step(float* h, const void* y, DType y_dtype, const float* w, float eps, const float* taps, int K, int state_offset,
                                     StepContext& ctx, void* out) {
@@ -102,11 +110,12 @@ inline void rotate_slice(const void* src, long long src_ld, int src_head, int sr
 
 // the heads' products of a step of few tokens in bfloat16, with the gate or the rotated tail that follows them (csrc/head_products.cu)
 inline void head_products_few(const void* x, long long x_ld, int x_head, const void* w, long long w_head, bool k_by_n, void* out, long long out_ld,
-                              int out_head, int N, int K, int H, const float* gate, long long gate_ld, int tail, const RotaryTable* rot,
+                              int out_head, int N, int K, int H, const float* gate, long long gate_ld, bool gate_per_head, int tail, const RotaryTable* rot,
                               const StepContext& ctx) {
     Timed t("head_products_few", ctx.stream);
     const bool turns = tail > 0 && rot && rot->inv_freq;
-    check(vm_head_products_few(x, x_ld, x_head, w, w_head, k_by_n ? 1 : 0, out, out_ld, out_head, ctx.T, N, K, H, gate, gate_ld, tail, ctx.positions,
+    check(vm_head_products_few(x, x_ld, x_head, w, w_head, k_by_n ? 1 : 0, out, out_ld, out_head, ctx.T, N, K, H, gate, gate_ld, gate_per_head ? 1 : 0, tail,
+                               ctx.positions,
                                turns ? rot->inv_freq : nullptr, turns ? rot->rotary_dim : 0, turns ? rot->pairing : 0, ctx.stream),
           "head_products_few", ctx.stream);
 }
@@ -166,6 +175,21 @@ inline void latent_rope_norm_write(const float* down, int ld, int q_rank, int kv
                                     write ? kv.k_pages : nullptr, write ? kv.n_pages : 0, rot_dim, rot.inv_freq ? rot.rotary_dim : 0, rot.inv_freq,
                                     rot.pairing, ctx.T, code(ctx.act_dtype), ctx.err, ctx.stream),
           "latent_norm_write", ctx.stream);
+}
+
+// directly projected queries: their unrotated parts to q, their turned parts behind each head's room of q_far; latent and key part to the cache
+inline void latent_direct(const float* proj, int ld, int H, int D, int R, int kv_rank, const float* wkv, float eps, void* q, void* q_far,
+                          const StepContext& ctx, const KVView& kv, bool write, const RotaryTable& rot) {
+    Timed t("latent_direct", ctx.stream);
+    check(vm_latent_direct(proj, ld, H, D, R, kv_rank, wkv, eps, q, q_far, ctx.positions, ctx.seq_of_token, kv.block_table, kv.table_width,
+                           write ? kv.k_pages : nullptr, write ? kv.n_pages : 0, rot.inv_freq ? rot.rotary_dim : 0, rot.inv_freq, rot.pairing, ctx.T,
+                           code(ctx.act_dtype), ctx.err, ctx.stream),
+          "latent_direct", ctx.stream);
+}
+
+inline void soft_cap(float* x, long long n, float cap, cudaStream_t s) {
+    Timed t("soft_cap", s);
+    check(vm_soft_cap(x, n, cap, s), "soft_cap", s);
 }
 
 constexpr int MLSTM_SCAN_MAX_TOKENS = 8;
@@ -272,6 +296,7 @@ struct BiasedMask {
     const int* bucket_of = nullptr;     // device int32 [far + 1]
     int far = 0, rows = 0, window = 0, keep_first = 0;
     const float* sink = nullptr;        // device float32 [H], or null: exp(sink[h]) joins head h's softmax denominator
+    const float* slopes = nullptr;      // device float32 [H], or null: slopes[h] (i - j) comes off head h's score of key j at place i
     int v_row_stride = 0;               // elements between neighbouring tokens' value rows (0: Dv); Dk with the key pool as value pool: values inside keys
 };
 // attention of the step's tokens over the cache with that mask and bias; keys of Dk, values of Dv; picks the kernel by shape and dtype
@@ -467,8 +492,9 @@ struct PrepareArgs {
     const float *q_norm = nullptr, *k_norm = nullptr;
     float eps = 0.f;
     RotaryTable rot;
-    int H = 0, G = 0, Dk = 0, Dv = 0;
+    int H = 0, G = 0, Dk = 0, Dv = 0;   // G = 0: a row of queries alone
     bool values_are_keys = false;
+    bool unit_heads = false;            // every q and k head divided by its root mean square
 };
 inline void mixer_prepare(const float* proj, int ld, const PrepareArgs& a, StepContext& ctx, const KVView& kv, void* q_out) {
     Timed t("mixer_prepare", ctx.stream);
@@ -477,7 +503,7 @@ inline void mixer_prepare(const float* proj, int ld, const PrepareArgs& a, StepC
     check(vm_mixer_prepare(proj, ld, a.bias, a.taps, a.K, ctx.state(), ctx.state_floats(), ctx.state_offset, a.q_norm, a.k_norm, a.eps, a.rot.inv_freq,
                            a.rot.rotary_dim, a.rot.pairing, ctx.positions, ctx.seq_of_token, ctx.cu_tokens, ctx.slots, kv.block_table, kv.table_width, q_out,
                            kv.owns ? kv.k_pages : nullptr, kv.owns ? kv.v_pages : nullptr, kv.owns ? kv.n_pages : 0, ctx.T, ctx.B, a.H, a.G, a.Dk, a.Dv,
-                           a.values_are_keys ? 1 : 0, ctx.one_token_each ? 1 : 0, code(ctx.act_dtype), ctx.err, ctx.stream),
+                           a.values_are_keys ? 1 : 0, a.unit_heads ? 1 : 0, ctx.one_token_each ? 1 : 0, code(ctx.act_dtype), ctx.err, ctx.stream),
           "mixer_prepare", ctx.stream);
     if (a.taps && a.K > 1 && !ctx.one_token_each) ++counters().own_launches;
 }
@@ -531,6 +557,61 @@ inline void decayed_memory(float* proj, int ld, const MemoryArgs& a, StepContext
 inline void memory_output(const float* o, const float* g, int ldg, const float* w, float eps, void* out, int T, int H, int Dv, DType act, cudaStream_t s) {
     Timed t("memory_output", s);
     check(vm_memory_output(o, g, ldg, w, eps, out, T, H, Dv, code(act), s), "memory_output", s);
+}
+
+// the gated delta rule over the running part's state: from the projections (layout as vm_delta_step) to the gated, normed heads in `out`
+struct DeltaArgs {
+    int g_off = 0, b_off = 0, a_off = 0;
+    const float* taps = nullptr;        // float32 [2 G Dk + H Dv, K]
+    int K = 1;
+    const float *A_log = nullptr, *dt_bias = nullptr, *norm_w = nullptr;
+    float eps = 0.f, q_scale = 1.f;
+    int H = 0, G = 0, Dk = 0, Dv = 0;
+};
+constexpr int DELTA_CHUNKS_FROM_TOKENS = 64;    // a step's capacity from which prompts run chunk by chunk
+inline void delta_rule(const float* proj, int ld, const DeltaArgs& a, StepContext& ctx, void* out) {
+    need_state(ctx, vm_delta_state_floats(a.H, a.G, a.Dk, a.Dv, a.K), "delta_rule");
+    // The choice follows the step's capacity bucket alone, so that every step of a bucket asks for the same scratch: decode steps take one
+    // launch, the smallest pieces go token by token, everything else chunk by chunk (every sequence may end in a chunk that is not full).
+    if (ctx.one_token_each && vm_delta_step_fits(a.Dk, a.Dv) && a.Dk % 2 == 0 && ctx.state_floats() % 4 == 0 && ctx.state_offset % 4 == 0) {
+        Timed t("delta_step", ctx.stream);
+        check(vm_delta_step(proj, ld, a.g_off, a.b_off, a.a_off, a.taps, a.K, ctx.state(), ctx.state_floats(), ctx.state_offset, ctx.positions, ctx.slots, a.A_log,
+                            a.dt_bias, a.norm_w, a.eps, a.q_scale, out, ctx.B, a.H, a.G, a.Dk, a.Dv, code(ctx.act_dtype), ctx.stream),
+              "delta_step", ctx.stream);
+        return;
+    }
+    const long long C = 2ll * a.G * a.Dk + static_cast<long long>(a.H) * a.Dv;
+    float* rows = static_cast<float*>(ctx.take_tokens(C, DType::F32));
+    float* gates = static_cast<float*>(ctx.take_tokens(2ll * a.H, DType::F32));
+    {
+        Timed t("delta_prepare", ctx.stream);
+        check(vm_delta_prepare(proj, ld, a.b_off, a.a_off, a.taps, a.K, ctx.state(), ctx.state_floats(), ctx.state_offset, ctx.positions, ctx.seq_of_token,
+                               ctx.cu_tokens, ctx.slots, a.A_log, a.dt_bias, a.q_scale, rows, gates, ctx.T, ctx.B, a.H, a.G, a.Dk, a.Dv, ctx.stream),
+              "delta_prepare", ctx.stream);
+        if (a.K > 1) ++counters().own_launches;
+    }
+    float* o = static_cast<float*>(ctx.take_tokens(static_cast<long long>(a.H) * a.Dv, DType::F32));
+    const int chunk = vm_delta_chunk_tokens(a.Dk, a.Dv);
+    if (chunk > 0 && !ctx.one_token_each && ctx.T_cap >= DELTA_CHUNKS_FROM_TOKENS) {
+        Timed t("delta_chunks", ctx.stream);
+        float* scratch = static_cast<float*>(ctx.take(vm_delta_scratch_floats(ctx.T_cap / chunk + ctx.B_cap, a.H, a.Dk, a.Dv), DType::F32));
+        int n_chunks = 0;
+        for (int b = 0; b < ctx.B; ++b) n_chunks += (ctx.host_cu_tokens[b + 1] - ctx.host_cu_tokens[b] + chunk - 1) / chunk;
+        check(vm_delta_chunks(rows, gates, ctx.state(), ctx.state_floats(), ctx.state_offset, ctx.cu_tokens, ctx.slots, o, scratch, n_chunks, ctx.T, ctx.B, a.H, a.G,
+                              a.Dk, a.Dv, ctx.stream),
+              "delta_chunks", ctx.stream);
+        counters().own_launches += 2;       // three kernels
+        ctx.give(scratch);
+    } else {
+        Timed t("delta_scan", ctx.stream);
+        check(vm_delta_scan(rows, gates, ctx.state(), ctx.state_floats(), ctx.state_offset, ctx.cu_tokens, ctx.slots, o, ctx.T, ctx.B, a.H, a.G, a.Dk, a.Dv,
+                            ctx.stream),
+              "delta_scan", ctx.stream);
+    }
+    memory_output(o, proj + a.g_off, ld, a.norm_w, a.eps, out, ctx.T, a.H, a.Dv, ctx.act_dtype, ctx.stream);
+    ctx.give(o);
+    ctx.give(gates);
+    ctx.give(rows);
 }
 
 int sm_count();                     // streaming multiprocessors of the current device, asked once

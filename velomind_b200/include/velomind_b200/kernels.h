@@ -85,7 +85,7 @@ int vm_sigmoid_gate(void* x, const float* gate, long long gate_ld, int T, int co
 // [K, N] (k_by_n) or [N, K]; with [N, K] an optional gate (out *= sigmoid(gate[t, h * N + n]), float32 rows), with [K, N] an optional tail
 // (out[t, h, N : N + tail] = x[t, h, K : K + tail], its first rotary_dim values turned by the token's position)
 int vm_head_products_few(const void* x, long long x_ld, int x_head, const void* w, long long w_head, int k_by_n, void* out, long long out_ld,
-                         int out_head, int T, int N, int K, int H, const float* gate, long long gate_ld, int tail, const int* positions,
+                         int out_head, int T, int N, int K, int H, const float* gate, long long gate_ld, int gate_per_head, int tail, const int* positions,
                          const float* inv_freq, int rotary_dim, int pairing, cudaStream_t stream);
 
 // ---- mlstm.cu: the matrix-memory recurrence with its output stage
@@ -156,16 +156,16 @@ int vm_attention_biased_generic(const void* q, int q_row_stride, const void* kpa
 // more term of head h's softmax denominator, without a key or a value, not scaled.  v_row_stride: elements between the value rows of
 // neighbouring tokens in `vpages` (0: Dv); with vpages == kpages and v_row_stride == Dk a token's value is the first Dv values of its key row.
 int vm_attention_sink_generic(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
-                              const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, const float* sink,
+                              const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, const float* sink, const float* slopes,
                               int v_row_stride, void* out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
                               int n_pages, int act_dtype, int* err, cudaStream_t stream);
 int vm_attention_sink_prefill_fits(int Dk, int Dv, int values_in_keys);
 int vm_attention_sink_prefill_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                                    const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel, const int* bucket_of, int far,
-                                   int rel_rows, const float* sink, int v_row_stride, void* out, int H, int Hkv, int Dk, int Dv, float scale, int window,
+                                   int rel_rows, const float* sink, const float* slopes, int v_row_stride, void* out, int H, int Hkv, int Dk, int Dv, float scale, int window,
                                    int keep_first, int n_pages, int* err, cudaStream_t stream);
 int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
-                                  const int* positions, const float* rel, const int* bucket_of, int far, const float* sink, int v_row_stride, void* out,
+                                  const int* positions, const float* rel, const int* bucket_of, int far, const float* sink, const float* slopes, int v_row_stride, void* out,
                                   int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err,
                                   cudaStream_t stream);
 
@@ -282,7 +282,7 @@ int vm_embed_pairs(const void* table, const void* pairs, int table_dtype, const 
 int vm_mixer_prepare(const float* proj, int ld, const float* bias, const float* taps, int K, float* state, long long state_stride, int state_offset,
                      const float* q_norm, const float* k_norm, float eps, const float* inv_freq, int rotary_dim, int pairing, const int* positions,
                      const int* seq_of_token, const int* cu_tokens, const int* slots, const int* block_table, int max_blocks, void* q_out, void* kpages,
-                     void* vpages, int n_pages, int T, int B, int H, int G, int Dk, int Dv, int values_are_keys, int one_token_each, int act_dtype,
+                     void* vpages, int n_pages, int T, int B, int H, int G, int Dk, int Dv, int values_are_keys, int unit_heads, int one_token_each, int act_dtype,
                      int* err, cudaStream_t stream);
 // x[t, c] *= sigmoid(g[t, c / per]), g float32 rows of stride ldg: one gate for every `per` neighbouring values (a head)
 int vm_sigmoid_gate_heads(void* x, const float* g, int ldg, int T, int cols, int per, int act_dtype, cudaStream_t stream);
@@ -323,6 +323,40 @@ void* vm_event_create(void);
 int vm_event_destroy(void* event);
 int vm_event_synchronize(void* event);
 int vm_upload_record(void* dst, const void* src, long long nbytes, void* event, cudaStream_t stream);
+
+// ---- sublayer.cu, latent_cache.cu, elementwise.cu: what layers with a norm on both sides of a sublayer, latent attention with directly projected
+// queries, and a head with capped logits need
+// h float32 [T, hid] += rmsnorm(y + bias) * w_out; out [T, hid] = rmsnorm(h) * w_in (y, out in act_dtype; bias float32 [hid] or null).  With
+// `rows` (int32 [n]) only those rows are made, into rows 0 .. n of out, and h is not written; else n = T
+int vm_norm_sum_norm(float* h, const void* y, const float* bias, const float* w_out, float eps_out, const float* w_in, float eps_in, void* out,
+                     const int* rows, int n, int hid, int act_dtype, cudaStream_t stream);
+// proj float32 [T, ld]: H queries of D unrotated and R rotated values, a latent of kv_rank, a key part of R for all heads; q [T, H D];
+// q_far [T, H (kv_rank + R)] receives every head's turned part behind its kv_rank; pages [n_pages, VM_PAGE_TOKENS, kv_rank + R] (null: none written)
+int vm_latent_direct(const float* proj, int ld, int H, int D, int R, int kv_rank, const float* wkv, float eps, void* q, void* q_far,
+                     const int* positions, const int* seq_of_token, const int* block_table, int max_blocks, void* pages, int n_pages, int rotary_dim,
+                     const float* inv_freq, int pairing, int T, int act_dtype, int* err, cudaStream_t stream);
+int vm_soft_cap(float* x, long long n, float cap, cudaStream_t stream);      // x <- cap tanh(x / cap), in place
+
+// ---- delta_rule.cu: the gated delta rule, S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, behind short convolutions with SiLU and
+// unit vectors.  proj float32 [T, ld]: q (G Dk columns), k (G Dk), v (H Dv) first, then wherever the offsets say: the SiLU gate's H Dv columns
+// (g_off), beta's and the decay's logits (b_off, a_off, H each).  taps float32 [2 G Dk + H Dv, K].  A sequence keeps
+// vm_delta_state_floats words at state_offset of its row of `state` (zero at its start).
+int vm_delta_state_floats(int H, int G, int Dk, int Dv, int K);
+// one token per sequence, one launch: out [B, H Dv] = o / rms(o) norm_w silu(gate) in act_dtype
+int vm_delta_step_fits(int Dk, int Dv);
+int vm_delta_step(const float* proj, int ld, int g_off, int b_off, int a_off, const float* taps, int K, float* state, long long state_stride,
+                  int state_offset, const int* positions, const int* slots, const float* A_log, const float* dt_bias, const float* norm_w, float eps,
+                  float q_scale, void* out, int B, int H, int G, int Dk, int Dv, int act_dtype, cudaStream_t stream);
+// the general way: the preparation (rows float32 [T, 2 G Dk + H Dv], gates float32 [T, 2 H]: beta, log g), then one of the two below (o float32 [T, H Dv])
+int vm_delta_prepare(const float* proj, int ld, int b_off, int a_off, const float* taps, int K, float* state, long long state_stride, int state_offset,
+                     const int* positions, const int* seq_of_token, const int* cu_tokens, const int* slots, const float* A_log, const float* dt_bias,
+                     float q_scale, float* rows, float* gates, int T, int B, int H, int G, int Dk, int Dv, cudaStream_t stream);
+int vm_delta_scan(const float* rows, const float* gates, float* state, long long state_stride, int state_offset, const int* cu_tokens, const int* slots,
+                  float* o, int T, int B, int H, int G, int Dk, int Dv, cudaStream_t stream);
+int vm_delta_chunk_tokens(int Dk, int Dv);           // tokens per chunk of vm_delta_chunks (0: it does not take these sizes)
+long long vm_delta_scratch_floats(int n_chunks, int H, int Dk, int Dv);
+int vm_delta_chunks(const float* rows, const float* gates, float* state, long long state_stride, int state_offset, const int* cu_tokens, const int* slots,
+                    float* o, float* scratch, int n_chunks, int T, int B, int H, int G, int Dk, int Dv, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -278,7 +278,9 @@ public:
     DType dtype;                               // the engine's activation dtype: F32 or BF16
     cudaStream_t stream;
     DeviceTensor upload(const HostTensor& t, DType as);
-    DeviceTensor upload_stacked(const std::vector<const HostTensor*>& parts, DType as);   // rows of several matrices, one tensor
+    // rows of several matrices, one tensor; its rows are filled up with zeros to a multiple of `row_multiple`
+    DeviceTensor upload_stacked(const std::vector<const HostTensor*>& parts, DType as, int row_multiple = 1);
+    DeviceTensor upload_scaled(const HostTensor& t, float factor);                         // float32, every value times `factor`
     DeviceTensor upload_floats(const std::vector<float>& values);
     DeviceTensor upload_ints(const std::vector<int>& values);
     // dtype a weight matrix is kept in: the compute dtype, except that a tensor stored in 32-bit stays 32-bit
@@ -479,6 +481,14 @@ struct StepContext {
     // (a layer whose norm sits on its sublayers' outputs leaves that norm to whoever adds the delta)
     const float* pending_norm_weight = nullptr;
     float pending_norm_eps = 0.f;
+    // A mixer whose output product has a bias may leave that bias to a wiring that can take it along when it adds the mixer's result: the
+    // wiring says so with `takes_row_bias` before it runs the mixer, and finds the bias (float32 [hidden], or null) in `row_bias` afterwards.
+    bool takes_row_bias = false;
+    const float* row_bias = nullptr;
+    bool leave_row_bias(const float* bias) {
+        if (takes_row_bias) row_bias = bias;
+        return takes_row_bias;
+    }
     // ... or, in a model with several copies of the stream, through the mixing its layer left with it: copy t becomes
     // sum_s pending_mix[s, t] x_s + pending_out[t] * delta (device float32 [streams, streams] and [streams])
     const float *pending_mix = nullptr, *pending_out = nullptr;
@@ -537,6 +547,8 @@ public:
 
 class Mixer : public Part {
 public:
+    // what the mixer keeps per sequence; for a mixer that reads another run's cache, what it must still find there (the run that keeps it
+    // then keeps as much as any of its readers asks for)
     virtual CacheNeed cache_need() const { return {}; }
     virtual void forward(StepContext& ctx, const void* x, void* out) = 0;       // x, out [T, hid] activation dtype
     // optional: take the norm before the part and the residual sum after it into the part's own kernels

@@ -254,6 +254,90 @@ private:
     DeviceTensor in_[2], out_[2], mix_[2];
 };
 
+// A norm on both sides of every sublayer: h += share * norm_out(sublayer(norm_in(h))).  The norms in front are the layer's own parts, those
+// behind are tensors of the wiring (`mixer_out`, `feed_forward_out`, [hidden]); `share` is multiplied into their weights when they are
+// bound.  A sublayer's sum and the next one's norm are one kernel: a layer leaves its last result pending with the norm it joins the
+// stream through, and whoever comes next (a layer, or the model's final norm) takes it along.
+class BothNormsBlock : public Arrangement {
+public:
+    BothNormsBlock(const BlockParts& p, int hidden, double eps, double share, std::string mixer_out, std::string ff_out, bool feed_forward)
+        : p_(p), hidden_(hidden), eps_(static_cast<float>(eps)), share_(static_cast<float>(share)), mixer_out_(std::move(mixer_out)), ff_out_(std::move(ff_out)),
+          feed_forward_(feed_forward) {
+        if (hidden <= 0) throw ConfigError("arrangement 'both_norms': argument 'hidden' must be positive");
+        if (mixer_out_.empty() || (feed_forward_ && ff_out_.empty())) throw ConfigError("arrangement 'both_norms': the norms behind the sublayers need their tensors' names");
+    }
+    bool graph_safe() const override { return true; }
+
+    WeightTable weight_specs() const override {
+        WeightTable t;
+        t[mixer_out_].shape = {hidden_};
+        t[mixer_out_].init_ones = true;
+        if (feed_forward_) {
+            t[ff_out_].shape = {hidden_};
+            t[ff_out_].init_ones = true;
+        }
+        return t;
+    }
+    void bind(const Weights& w, BindContext& bc) override {
+        out_[0] = bc.upload_scaled(w.at(mixer_out_), share_);
+        if (feed_forward_) out_[1] = bc.upload_scaled(w.at(ff_out_), share_);
+    }
+
+    void* forward(StepContext& ctx, float* h, void* pending) override {
+        if (ctx.hidden != hidden_) throw ConfigError("arrangement 'both_norms': the stream's width is not the one it was built for");
+        void* x = ctx.take_tokens(hidden_, ctx.act_dtype);
+        const float* nw = nullptr;
+        float eps = 0.f;
+        if (pending && ctx.pending_norm_weight && p_.mixer_norm->as_rms(&nw, &eps)) {
+            ops::norm_sum_norm(h, pending, nullptr, ctx.pending_norm_weight, ctx.pending_norm_eps, nw, eps, x, nullptr, ctx.T, hidden_, ctx.act_dtype, ctx.stream);
+            ctx.pending_norm_weight = nullptr;
+            ctx.give(pending);
+        } else {
+            if (ctx.pending_norm_weight) {
+                settle_pending(ctx, h, pending, hidden_);
+                pending = nullptr;
+            }
+            p_.mixer_norm->forward(ctx, h, pending, x, nullptr, 0);
+            ctx.give(pending);
+        }
+        void* y = ctx.take_tokens(hidden_, ctx.act_dtype);
+        const bool joins = feed_forward_ && p_.feed_forward_norm->as_rms(&nw, &eps);
+        ctx.takes_row_bias = joins;                        // (this wiring's sum with the next norm takes the output product's bias along)
+        p_.mixer->forward(ctx, x, y);
+        const float* bias = ctx.row_bias;
+        ctx.takes_row_bias = false;
+        ctx.row_bias = nullptr;
+        ctx.give(x);
+        if (!feed_forward_) return leave(ctx, y, 0);
+        x = ctx.take_tokens(hidden_, ctx.act_dtype);
+        const float* w0 = static_cast<const float*>(out_[0].ptr);
+        if (joins) {
+            ops::norm_sum_norm(h, y, bias, w0, eps_, nw, eps, x, nullptr, ctx.T, hidden_, ctx.act_dtype, ctx.stream);
+        } else {
+            ops::norm_residual_add(h, y, hidden_, ctx.act_dtype, w0, eps_, ctx.T, hidden_, ctx.stream);
+            p_.feed_forward_norm->forward(ctx, h, nullptr, x, nullptr, 0);
+        }
+        ctx.give(y);
+        y = ctx.take_tokens(hidden_, ctx.act_dtype);
+        p_.feed_forward->forward(ctx, x, y);
+        ctx.give(x);
+        return leave(ctx, y, 1);
+    }
+
+private:
+    void* leave(StepContext& ctx, void* y, int which) {
+        ctx.pending_norm_weight = static_cast<const float*>(out_[which].ptr);
+        ctx.pending_norm_eps = eps_;
+        return y;
+    }
+    BlockParts p_;
+    int hidden_;
+    float eps_, share_;
+    std::string mixer_out_, ff_out_;
+    bool feed_forward_;
+    DeviceTensor out_[2];
+};
+
 // The feed-forward of a layer that has none: no weights, never run.
 class NoFeedForward : public FeedForward {
 public:
@@ -280,6 +364,13 @@ struct Reg {
             return std::make_shared<HyperConnections>(parts, static_cast<int>(arg_int(a, "hidden", k)), static_cast<int>(arg_int(a, "streams", k)),
                                                       arg_string_or(a, "mixer_tensors", "hc1", k), arg_string_or(a, "feed_forward_tensors", "hc2", k),
                                                       arg_int_or(a, "feed_forward", 1, k) != 0);
+        });
+        // a norm in front of and behind every sublayer
+        register_arrangement("both_norms", [](const json::Value& a, const BlockParts& parts) {
+            const char* k = "both_norms";
+            return std::make_shared<BothNormsBlock>(parts, static_cast<int>(arg_int(a, "hidden", k)), arg_number(a, "eps", k), arg_number_or(a, "share", 1.0, k),
+                                                    arg_string_or(a, "mixer_out", "norm1b", k), arg_string_or(a, "feed_forward_out", "norm2b", k),
+                                                    arg_int_or(a, "feed_forward", 1, k) != 0);
         });
         register_part("feed_forward", "none", [](const json::Value&) { return std::make_shared<NoFeedForward>(); });
     }

@@ -61,11 +61,11 @@ private:
 
 // logits = x W^T in float32.  `tied_to` names the tensor that stands in when the checkpoint has no head of its own
 // (examples/smollm2/model_loader.cpp:124-158: lm_head.weight if present, else the embedding when tied); the device tensor is
-// then shared with the embedding, not copied.
+// then shared with the embedding, not copied.  `soft_cap` c > 0: logits <- c tanh(logits / c).
 class LinearHead : public Head {
 public:
-    LinearHead(int vocab, int hidden, std::string tied_to, std::string tensor = "weight")
-        : vocab_(vocab), hidden_(hidden), tied_to_(std::move(tied_to)), tensor_(std::move(tensor)) {}
+    LinearHead(int vocab, int hidden, std::string tied_to, std::string tensor = "weight", float soft_cap = 0.f)
+        : vocab_(vocab), hidden_(hidden), tied_to_(std::move(tied_to)), tensor_(std::move(tensor)), cap_(soft_cap) {}
     WeightTable weight_specs() const override {
         WeightTable t;
         t[tensor_].shape = {vocab_, hidden_};
@@ -79,11 +79,13 @@ public:
             ops::skinny_linear(x, nullptr, 0.f, proj_.weight, ctx.R, logits, vocab_, true, nullptr, ctx.err, ctx.stream);   // few rows: stream the table once
         else
             proj_.apply(ctx, x, ctx.act_dtype, logits, DType::F32, ctx.R, ctx.R_cap);
+        if (cap_ > 0.f) ops::soft_cap(logits, static_cast<long long>(ctx.R) * vocab_, cap_, ctx.stream);
     }
 
 private:
     int vocab_, hidden_;
     std::string tied_to_, tensor_;
+    float cap_;
     Linear proj_;
 };
 
@@ -101,7 +103,8 @@ RegisterPart reg_pairs("embedding", "token_pairs_table", [](const json::Value& a
 });
 RegisterPart reg_head("head", "linear", [](const json::Value& a) {
     return std::make_shared<LinearHead>(static_cast<int>(arg_int(a, "vocab", "linear")), static_cast<int>(arg_int(a, "hidden", "linear")),
-                                        arg_string_or(a, "tied_to", "", "linear"), arg_string_or(a, "tensor", "weight", "linear"));
+                                        arg_string_or(a, "tied_to", "", "linear"), arg_string_or(a, "tensor", "weight", "linear"),
+                                        static_cast<float>(arg_number_or(a, "soft_cap", 0.0, "linear")));
 });
 }  // namespace
 

@@ -6,8 +6,12 @@
 //       the K - 1 last projected rows of a sequence are part of its state
 //   `values_are_keys`: there is no W_v; a token's value is its key as it leaves the convolution, before norm and rotation
 //   `qk_norm`: RMS norm over the whole projection of q (and of k), all heads at once, with a weight per column (q.norm, k.norm)
+//   `unit_heads`: every q and k head divided by its root mean square over `dim` (a norm without a weight)
 //   `position`: rotary positions on the first rotary_dim values of every q and k head, either pairing
 //   score(i, j) = scale q_i . k_j;  i sees j  iff  j <= i and (window == 0 or i - j < window or j < keep_first)
+//   `slopes`: 2^(-8 (h + 1) / H) (i - j) comes off head h's score of key j
+//   `own_kv` = 0: the layer has no k and v of its own; its schedule entry names the run whose keys and values (as cached) it reads, with its
+//       own queries, window and everything else
 //   `sink`: exp(sink_h), a learned number per head, joins head h's softmax denominator without a key or a value
 //   `gate`: "values": the heads' outputs times sigmoid(W_g x) value by value ([H vdim, hidden]); "heads": one gate per head ([H, hidden])
 //   then W_o, with the bias o.b if `out_bias`
@@ -40,6 +44,9 @@ public:
         qk_norm_ = arg_int_or(a, "qk_norm", 0, k) != 0;
         sink_ = arg_int_or(a, "sink", 0, k) != 0;
         values_are_keys_ = arg_int_or(a, "values_are_keys", 0, k) != 0;
+        unit_heads_ = arg_int_or(a, "unit_heads", 0, k) != 0;
+        slopes_ = arg_int_or(a, "slopes", 0, k) != 0;
+        own_ = arg_int_or(a, "own_kv", 1, k) != 0;
         eps_ = static_cast<float>(arg_number_or(a, "eps", 1e-6, k));
         const std::string gate = arg_string_or(a, "gate", "none", k);
         if (gate != "none" && gate != "values" && gate != "heads") throw ConfigError(format("part '%s': gate is \"none\", \"values\" or \"heads\"", k));
@@ -51,22 +58,26 @@ public:
         if (window_ < 0 || keep_first_ < 0) throw ConfigError(format("part '%s': window and keep_first must not be negative", k));
         if (window_ == 0) keep_first_ = 0;
         if (K_ < 0 || K_ > 16) throw ConfigError(format("part '%s': taps (%d) must be within 0..16", k, K_));
+        if (qk_norm_ && unit_heads_) throw ConfigError(format("part '%s': qk_norm and unit_heads exclude each other", k));
+        if (!own_ && (K_ >= 1 || values_are_keys_ || qk_norm_))
+            throw ConfigError(format("part '%s': a layer without keys of its own takes no convolution, no values that are keys and no norm over the projections", k));
         if (const json::Value* pos = a.find("position")) position_ = build_part_as<Position>("position", part_spec_from_json(*pos, "general_attention.position"));
     }
 
-    long long row_cols() const { return static_cast<long long>(H_ + G_) * Dk_ + (values_are_keys_ ? 0 : static_cast<long long>(G_) * Dv_); }
+    bool has_v() const { return own_ && !values_are_keys_; }
+    long long row_cols() const { return static_cast<long long>(H_ + (own_ ? G_ : 0)) * Dk_ + (has_v() ? static_cast<long long>(G_) * Dv_ : 0); }
     long long proj_cols() const { return row_cols() + gate_cols_; }
 
     WeightTable weight_specs() const override {
         WeightTable t;
         t["q"].shape = {static_cast<long long>(H_) * Dk_, hidden_};
-        t["k"].shape = {static_cast<long long>(G_) * Dk_, hidden_};
-        if (!values_are_keys_) t["v"].shape = {static_cast<long long>(G_) * Dv_, hidden_};
+        if (own_) t["k"].shape = {static_cast<long long>(G_) * Dk_, hidden_};
+        if (has_v()) t["v"].shape = {static_cast<long long>(G_) * Dv_, hidden_};
         t["o"].shape = {hidden_, static_cast<long long>(H_) * Dv_};
         if (bias_) {
             t["q.b"].shape = {static_cast<long long>(H_) * Dk_};
-            t["k.b"].shape = {static_cast<long long>(G_) * Dk_};
-            if (!values_are_keys_) t["v.b"].shape = {static_cast<long long>(G_) * Dv_};
+            if (own_) t["k.b"].shape = {static_cast<long long>(G_) * Dk_};
+            if (has_v()) t["v.b"].shape = {static_cast<long long>(G_) * Dv_};
         }
         if (out_bias_) t["o.b"].shape = {hidden_};
         if (K_ >= 1) {
@@ -85,13 +96,14 @@ public:
     }
 
     void bind(const Weights& w, BindContext& bc) override {
-        std::vector<const HostTensor*> stacked = {&w.at("q"), &w.at("k")}, biases, taps;
-        if (!values_are_keys_) stacked.push_back(&w.at("v"));
+        std::vector<const HostTensor*> stacked = {&w.at("q")}, biases, taps;
+        if (own_) stacked.push_back(&w.at("k"));
+        if (has_v()) stacked.push_back(&w.at("v"));
         if (gate_cols_) stacked.push_back(&w.at("g"));
         proj_.bind(stacked, bc);
         out_.bind({&w.at("o")}, bc);
         const char* parts[3] = {"q", "k", "v"};
-        for (int i = 0; i < (values_are_keys_ ? 2 : 3); ++i) {
+        for (int i = 0; i < (has_v() ? 3 : (own_ ? 2 : 1)); ++i) {
             if (bias_) biases.push_back(&w.at(std::string(parts[i]) + ".b"));
             if (K_ >= 1) taps.push_back(&w.at(std::string(parts[i]) + ".conv"));
         }
@@ -103,6 +115,11 @@ public:
             wk_ = bc.upload(w.at("k.norm"), DType::F32);
         }
         if (sink_) sinks_ = bc.upload(w.at("sink"), DType::F32);
+        if (slopes_) {
+            std::vector<float> s;
+            for (int h = 0; h < H_; ++h) s.push_back(static_cast<float>(std::exp2(-8.0 * (h + 1) / H_)));
+            slope_ = bc.upload_floats(s);
+        }
         if (position_) rotary_ = position_->tables(bc);
         if (rotary_.inv_freq && rotary_.rotary_dim > Dk_) throw ConfigError("part 'general_attention': the rotation covers more values than a head has");
     }
@@ -127,6 +144,7 @@ public:
         float* proj = static_cast<float*>(ctx.take_tokens(ld, DType::F32));
         project_f32(ctx, proj_, x, proj);
         const KVView kv = ctx.kv();
+        if (kv.owns != own_) throw ConfigError("an attention layer and its schedule disagree about whose keys and values it reads");
         ops::PrepareArgs p;
         p.bias = bias_ ? static_cast<const float*>(b_.ptr) : nullptr;
         p.taps = K_ >= 1 ? static_cast<const float*>(taps_.ptr) : nullptr;
@@ -136,7 +154,8 @@ public:
         p.eps = eps_;
         p.rot = rotary_;
         p.H = H_;
-        p.G = G_;
+        p.G = own_ ? G_ : 0;
+        p.unit_heads = unit_heads_;
         p.Dk = Dk_;
         p.Dv = Dv_;
         p.values_are_keys = values_are_keys_;
@@ -147,6 +166,7 @@ public:
         mask.window = window_;
         mask.keep_first = keep_first_;
         mask.sink = sink_ ? static_cast<const float*>(sinks_.ptr) : nullptr;
+        mask.slopes = slopes_ ? static_cast<const float*>(slope_.ptr) : nullptr;
         ops::attention_biased(ctx, q, H_ * Dk_, kv, att, H_, G_, Dk_, Dv_, scale_, mask);
         ctx.give(q);
         if (gate_cols_ && gate_per_ == 1) ops::sigmoid_gate(att, proj + row_cols(), ld, ctx.T, H_ * Dv_, act, ctx.stream);
@@ -154,17 +174,18 @@ public:
         ctx.give(proj);
         project(ctx, out_, att, out);
         ctx.give(att);
-        if (out_bias_) ops::join_rows(out, nullptr, static_cast<const float*>(ob_.ptr), 1.f, 0.f, nullptr, nullptr, 0.f, out, ctx.T, hidden_, act, ctx.stream);
+        if (out_bias_ && !ctx.leave_row_bias(static_cast<const float*>(ob_.ptr)))
+            ops::join_rows(out, nullptr, static_cast<const float*>(ob_.ptr), 1.f, 0.f, nullptr, nullptr, 0.f, out, ctx.T, hidden_, act, ctx.stream);
     }
 
 private:
     int hidden_ = 0, H_ = 0, G_ = 0, Dk_ = 0, Dv_ = 0, window_ = 0, keep_first_ = 0, K_ = 0, gate_cols_ = 0, gate_per_ = 1;
     float scale_ = 1.f, eps_ = 1e-6f;
-    bool bias_ = false, out_bias_ = false, qk_norm_ = false, sink_ = false, values_are_keys_ = false;
+    bool bias_ = false, out_bias_ = false, qk_norm_ = false, sink_ = false, values_are_keys_ = false, unit_heads_ = false, slopes_ = false, own_ = true;
     std::shared_ptr<Position> position_;
     RotaryTable rotary_;
     Linear proj_, out_;
-    DeviceTensor b_, taps_, ob_, wq_, wk_, sinks_;
+    DeviceTensor b_, taps_, ob_, wq_, wk_, sinks_, slope_;
 };
 
 namespace {

@@ -14,8 +14,10 @@ struct Linear {
     DeviceTensor weight;
     long long out_features = 0, in_features = 0;
 
-    void bind(const std::vector<const HostTensor*>& stored, BindContext& bc) {
-        weight = bc.upload_stacked(stored, bc.matrix_dtype(stored));
+    // `row_multiple`: rows of zeros are added until their number is a multiple of it (the products' rows then start on aligned addresses
+    // whatever the matrices' sizes, and the weight-streaming kernels take them)
+    void bind(const std::vector<const HostTensor*>& stored, BindContext& bc, int row_multiple = 1) {
+        weight = bc.upload_stacked(stored, bc.matrix_dtype(stored), row_multiple);
         out_features = weight.rows();
         in_features = weight.cols();
     }

@@ -65,6 +65,7 @@ public:
     }
 
     void forward(StepContext& ctx, const void* x, void* out) override {
+        ctx.takes_row_bias = false;                       // (two results are joined first: neither may leave its bias to the wiring)
         const int base = ctx.state_offset;
         void* a = ctx.take_tokens(hidden_, ctx.act_dtype);
         left_->forward(ctx, x, a);
