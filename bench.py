@@ -343,6 +343,30 @@ def vozetar_config(z, x):
                        {"type": "parallel_2", "mixer": par2, "mlp": dense}, {"type": "parallel", "mixer": par, "mlp": moe}]}
 
 
+# ------------------------------------------------------------------------------------------------ --design zabozen
+# The same widths, four layers with a norm on both sides of every sublayer and a SiLU-gated unit each: windowed attention with slopes by
+# distance; latent attention with a rotated key part of 32 values and every earlier token visible; the gated delta rule; attention on the
+# first layer's keys with a wider window.  Beside it Fidizen (the same latent attention kernels behind a query latent, with a window, a sink
+# and routed experts), Vozetar (windowed attention and linear attention with a matrix memory side by side) and the Llama decoder at equal
+# width and depth.
+ZABOZEN_EXTRA = {
+    "w1024": dict(kv_heads=4, window=1024, reader_window=1536, rot_dim=32, delta_heads=8, delta_kv_heads=4, delta_dim=128, delta_vdim=128, conv=4),
+    "w2048": dict(kv_heads=8, window=1024, reader_window=1536, rot_dim=32, delta_heads=16, delta_kv_heads=8, delta_dim=128, delta_vdim=128, conv=4),
+}
+
+
+def zabozen_config(z, x):
+    att = {"heads": z["heads"], "kv_heads": x["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5}
+    lat = {"heads": z["heads"], "dim": z["dim"], "rot_dim": x["rot_dim"], "vdim": z["dim"], "kv_rank": z["kv_rank"],
+           "scale": (z["dim"] + x["rot_dim"]) ** -0.5, "rot": {"base": 10000.0, "dims": x["rot_dim"]}}
+    dlt = {"heads": x["delta_heads"], "kv_heads": x["delta_kv_heads"], "dim": x["delta_dim"], "vdim": x["delta_vdim"], "conv": x["conv"]}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    return {"architecture": "Zabozen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.8, "logit_softcap": 25.0,
+            "layers": [{"type": "attention", "mixer": dict(att, mask={"size": x["window"]}), "mlp": dense},
+                       {"type": "latent_attention", "mixer": lat, "mlp": dense}, {"type": "delta", "mixer": dlt, "mlp": dense},
+                       {"type": "attention", "mixer": dict(att, mask={"size": x["reader_window"]}, kv_from=0), "mlp": dense}]}
+
+
 def kogilix_attention_config(z):
     att = {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"], "scale": z["dim"] ** -0.5}
     moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["shared_ff"]}}
@@ -371,7 +395,7 @@ def op_table(vm, engine, entries):
 
 
 def design_arm(args):
-    """Prompt and decode throughput of a design (Kogilix, Semesun, Fidizen, Vozetar) at a few sizes, beside the library's other models at equal size."""
+    """Prompt and decode throughput of a design (Kogilix, Semesun, Fidizen, Vozetar, Zabozen) at a few sizes, beside the library's other models at equal size."""
     import numpy as np
     import velomind_b200 as vm
     T, B, prompt_len = 2048, 8, 512
@@ -386,6 +410,9 @@ def design_arm(args):
             models.insert(0, ("semesun", semesun_config(z, SEMESUN_EXTRA[name])))
         if args.design == "vozetar":
             models = [("vozetar", vozetar_config(z, VOZETAR_EXTRA[name])), ("semesun", semesun_config(z, SEMESUN_EXTRA[name])), ("llama", llama_config_like(z))]
+        if args.design == "zabozen":
+            models = [("zabozen", zabozen_config(z, ZABOZEN_EXTRA[name])), ("fidizen", fidizen_config(z, FIDIZEN_EXTRA[name])),
+                      ("vozetar", vozetar_config(z, VOZETAR_EXTRA[name])), ("llama", llama_config_like(z))]
         if args.design == "fidizen":
             models = [("fidizen", fidizen_config(z, FIDIZEN_EXTRA[name])), ("kogilix_attention", kogilix_attention_config(z)), ("llama", llama_config_like(z))]
         for which, cfg in models:
@@ -516,7 +543,7 @@ def main() -> int:
     ap.add_argument("--quick", action="store_true", help="skip the batch 1 / 64 points and the end-to-end run")
     ap.add_argument("--shape", default="135m", choices=sorted(SHAPES),
                     help="sizes of the random model: the benchmark's SmolLM2-135M (default), or the 360M / 1.7B shapes of the family")
-    ap.add_argument("--design", default="", choices=["", "kogilix", "semesun", "fidizen", "vozetar"],
+    ap.add_argument("--design", default="", choices=["", "kogilix", "semesun", "fidizen", "vozetar", "zabozen"],
                     help="instead of the benchmark: prompt and decode throughput of another design of the library at a few layer sizes, "
                          "beside the Llama decoder at equal size (one JSON line of its own)")
     args = ap.parse_args()
