@@ -521,12 +521,62 @@ __global__ void memory_output_kernel(const float* __restrict__ o, const float* _
     }
 }
 
+// the same for heads of a multiple of four values up to 256, 16-byte loads: a lane keeps its four (or eight) values between the two passes
+__device__ __forceinline__ void mo_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void mo_store4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<const unsigned*>(&a);
+    r.y = *reinterpret_cast<const unsigned*>(&b);
+    *reinterpret_cast<uint2*>(p) = r;
+}
+template <typename T>
+__global__ void __launch_bounds__(256)
+memory_output_vec_kernel(const float* __restrict__ o, const float* __restrict__ g, int ldg, const float* __restrict__ w, float eps, T* __restrict__ out,
+                         long long n_heads, int H, int Dv) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= n_heads) return;
+    const int lane = threadIdx.x & 31;
+    const long long t = item / H;
+    const int h = (int)(item - t * H);
+    float4 x[2], gv[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+        const int d = 4 * (lane + 32 * n);
+        x[n] = gv[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d >= Dv) continue;
+        x[n] = *reinterpret_cast<const float4*>(o + (size_t)item * Dv + d);
+        gv[n] = *reinterpret_cast<const float4*>(g + (size_t)t * ldg + (size_t)h * Dv + d);
+        ss += x[n].x * x[n].x + x[n].y * x[n].y + x[n].z * x[n].z + x[n].w * x[n].w;
+    }
+    const float inv = 1.0f / sqrtf(vm_warp_sum(ss) / (float)Dv + eps);
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+        const int d = 4 * (lane + 32 * n);
+        if (d >= Dv) continue;
+        const float4 ww = w ? *reinterpret_cast<const float4*>(w + d) : make_float4(1.f, 1.f, 1.f, 1.f);
+        const float4 y = gv[n];
+        mo_store4(out + (size_t)item * Dv + d, make_float4(x[n].x * inv * ww.x * (y.x / (1.0f + expf(-y.x))), x[n].y * inv * ww.y * (y.y / (1.0f + expf(-y.y))),
+                                                           x[n].z * inv * ww.z * (y.z / (1.0f + expf(-y.z))), x[n].w * inv * ww.w * (y.w / (1.0f + expf(-y.w)))));
+    }
+}
+
 VM_API int vm_memory_output(const float* o, const float* g, int ldg, const float* w, float eps, void* out, int T, int H, int Dv, int act_dtype,
                             cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || Dv <= 0) return VM_ERR_BAD_ARG;
     const long long n = (long long)T * H;
     const int grid = (int)((n + 7) / 8);
+    if (Dv % 4 == 0 && Dv <= 256 && ldg % 4 == 0 && ((uintptr_t)o | (uintptr_t)g | (uintptr_t)w | (uintptr_t)out) % 16 == 0) {
+        if (act_dtype == VM_F32) vm_launch_pdl(memory_output_vec_kernel<float>, dim3(grid), dim3(256), 0, stream, o, g, ldg, w, eps, (float*)out, n, H, Dv);
+        else if (act_dtype == VM_BF16)
+            vm_launch_pdl(memory_output_vec_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, o, g, ldg, w, eps, (__nv_bfloat16*)out, n, H, Dv);
+        else return VM_ERR_UNSUPPORTED;
+        return vm_launch_status();
+    }
     if (act_dtype == VM_F32) vm_launch_pdl(memory_output_kernel<float>, dim3(grid), dim3(256), 0, stream, o, g, ldg, w, eps, (float*)out, n, H, Dv);
     else if (act_dtype == VM_BF16) vm_launch_pdl(memory_output_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, o, g, ldg, w, eps, (__nv_bfloat16*)out, n, H, Dv);
     else return VM_ERR_UNSUPPORTED;

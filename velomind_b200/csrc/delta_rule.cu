@@ -88,6 +88,91 @@ delta_prepare_kernel(const float* __restrict__ proj, int ld, int b_off, int a_of
     }
 }
 
+// The same for heads of a multiple of four values and up to four taps: a warp makes one head of RUN neighbouring tokens, a lane four (or NQ
+// times four) neighbouring channels, with the K - 1 rows before the token carried along in registers, so that every row is loaded once and a
+// halo of K - 1 rows per run.  Warps of neighbouring heads lie side by side: they read neighbouring parts of the same rows.
+constexpr int RUN = 8;
+__device__ __forceinline__ float4 dr_fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
+
+template <int K, int NQ>
+__global__ void __launch_bounds__(PREP_THREADS)
+delta_prepare_run_kernel(const float* __restrict__ proj, int ld, int b_off, int a_off, const float* __restrict__ taps, const float* __restrict__ state,
+                         long long state_stride, int kept_offset, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
+                         const int* __restrict__ cu_tokens, const int* __restrict__ slots, const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                         float q_scale, float* __restrict__ rows, float* __restrict__ gates, int T, int H, int G, int Dk, int Dv) {
+    vm_pdl_launch_dependents();
+    const int units = 2 * G + H + 1, C = 2 * G * Dk + H * Dv, lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * (PREP_THREADS / 32) + (threadIdx.x >> 5);
+    const int run = (int)(item / units), unit = (int)(item - (long long)run * units), t0 = run * RUN;
+    if (t0 >= T) return;
+    if (unit == 2 * G + H) {                              // beta and log g of the run's tokens
+        vm_pdl_wait();
+        for (int i = lane; i < RUN * H; i += 32) {
+            const int t = t0 + i / H, h = i % H;
+            if (t >= T) break;
+            const float b = proj[(size_t)t * ld + b_off + h], a = proj[(size_t)t * ld + a_off + h];
+            gates[(size_t)t * 2 * H + h] = 1.0f / (1.0f + expf(-b));
+            gates[(size_t)t * 2 * H + H + h] = -expf(A_log[h]) * dr_softplus(a + dt_bias[h]);
+        }
+        return;
+    }
+    const bool is_qk = unit < 2 * G;
+    const int D = is_qk ? Dk : Dv, col = is_qk ? unit * Dk : 2 * G * Dk + (unit - 2 * G) * Dv;
+    float4 w[NQ][K];                                      // w[.][j]: tap j of the lane's four channels
+#pragma unroll
+    for (int n = 0; n < NQ; ++n) {
+        const int c = 4 * (lane + 32 * n);
+        const float* tp = taps + (size_t)(col + (c < D ? c : 0)) * K;
+#pragma unroll
+        for (int j = 0; j < K; ++j) w[n][j] = make_float4(tp[j], tp[K + j], tp[2 * K + j], tp[3 * K + j]);
+    }
+    vm_pdl_wait();
+    const float scale = unit < G ? q_scale : 1.0f;
+    float4 win[NQ][K > 1 ? K - 1 : 1];                    // win[.][j]: the projected row K - 1 - j places back
+    int seq_before = -1;
+    for (int t = t0; t < min(t0 + RUN, T); ++t) {
+        const int seq = seq_of_token[t];
+        if (K > 1 && seq != seq_before) {
+            const int in_step = t - cu_tokens[seq];
+            const float* kept = state + (size_t)slots[seq] * state_stride + kept_offset + (size_t)((positions[t] - in_step) & 1) * (K - 1) * C;
+#pragma unroll
+            for (int n = 0; n < NQ; ++n) {
+                const int c = 4 * (lane + 32 * n);
+#pragma unroll
+                for (int j = 0; j < K - 1; ++j) {
+                    const int back = K - 1 - j;
+                    const float* src = back <= in_step ? proj + (size_t)(t - back) * ld : kept + (size_t)(K - 1 - back + in_step) * C;
+                    win[n][j] = c < D ? *reinterpret_cast<const float4*>(src + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+            }
+            seq_before = seq;
+        }
+        float4 y[NQ];
+        float ss = 0.f;
+#pragma unroll
+        for (int n = 0; n < NQ; ++n) {
+            const int c = 4 * (lane + 32 * n);
+            const float4 x = c < D ? *reinterpret_cast<const float4*>(proj + (size_t)t * ld + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j < K - 1; ++j) v = dr_fma4(w[n][j], win[n][j], v);
+            v = dr_fma4(w[n][K - 1], x, v);
+#pragma unroll
+            for (int j = 0; j + 1 < K - 1; ++j) win[n][j] = win[n][j + 1];
+            if (K > 1) win[n][K > 1 ? K - 2 : 0] = x;
+            y[n] = make_float4(dr_silu(v.x), dr_silu(v.y), dr_silu(v.z), dr_silu(v.w));
+            if (c < D) ss += y[n].x * y[n].x + y[n].y * y[n].y + y[n].z * y[n].z + y[n].w * y[n].w;
+        }
+        float f = 1.0f;
+        if (is_qk) f = scale / sqrtf(vm_warp_sum(ss) + UNIT_EPS);
+#pragma unroll
+        for (int n = 0; n < NQ; ++n) {
+            const int c = 4 * (lane + 32 * n);
+            if (c < D) *reinterpret_cast<float4*>(rows + (size_t)t * C + col + c) = make_float4(y[n].x * f, y[n].y * f, y[n].z * f, y[n].w * f);
+        }
+    }
+}
+
 // grid (B, slices of the channels): the kept rows of a sequence move on by the step's tokens, from the copy of its first place to the copy
 // of the place behind its last token (they may be the same one: a thread owns its channel and reads before it writes)
 constexpr int MAX_TAPS = 16;
@@ -389,7 +474,7 @@ delta_local_kernel(const float* __restrict__ rows, const float* __restrict__ gat
     float* kT = sm;                          // [Dk][CP]
     float* part = kT + (size_t)Dk * CP;      // [2][64][64]; then A, transposed, in the first half
     __shared__ double b[CH];
-    __shared__ float beta[CH];
+    __shared__ float beta[CH], beta_eb[CH];
     vm_pdl_launch_dependents();
     vm_pdl_wait();
     int start, len;
@@ -409,7 +494,9 @@ delta_local_kernel(const float* __restrict__ rows, const float* __restrict__ gat
     float* U = W + (size_t)Dk * CH;
     float* eb = U + (size_t)CH * Dv + (size_t)Dk * Dv;
     if (tid < CH) {
-        eb[tid] = expf((float)b[tid]);
+        const float e = expf((float)b[tid]);
+        beta_eb[tid] = beta[tid] * e;
+        eb[tid] = e;
         eb[CH + tid] = tid < len ? expf((float)(b[len - 1] - b[tid])) : 0.f;
     }
     __syncthreads();
@@ -419,10 +506,10 @@ delta_local_kernel(const float* __restrict__ rows, const float* __restrict__ gat
 #pragma unroll
             for (int t = 0; t < CH; t += 4) {
                 const float4 k = *reinterpret_cast<const float4*>(kT + col * CP + t);
-                x[t] = beta[t] * expf((float)b[t]) * k.x;
-                x[t + 1] = beta[t + 1] * expf((float)b[t + 1]) * k.y;
-                x[t + 2] = beta[t + 2] * expf((float)b[t + 2]) * k.z;
-                x[t + 3] = beta[t + 3] * expf((float)b[t + 3]) * k.w;
+                x[t] = beta_eb[t] * k.x;
+                x[t + 1] = beta_eb[t + 1] * k.y;
+                x[t + 2] = beta_eb[t + 2] * k.z;
+                x[t + 3] = beta_eb[t + 3] * k.w;
             }
         } else {
             const float* v = rows + (size_t)start * C + 2 * G * Dk + (size_t)h * Dv + (col - Dk);
@@ -702,10 +789,31 @@ VM_API int vm_delta_prepare(const float* proj, int ld, int b_off, int a_off, con
     const size_t smem = (size_t)PT * Dk * sizeof(float);
     if (smem > 96 * 1024 || 2 * G + H + 1 > 65535) return VM_ERR_UNSUPPORTED;
     const int kept = state_offset + H * Dk * Dv, C = 2 * G * Dk + H * Dv;
-    cudaError_t e = allow_smem(delta_prepare_kernel, smem);
-    if (e != cudaSuccess) return (int)e;
-    vm_launch_pdl(delta_prepare_kernel, dim3((T + PT - 1) / PT, 2 * G + H + 1), dim3(PREP_THREADS), smem, stream, proj, ld, b_off, a_off, taps, K,
-                  (const float*)state, state_stride, kept, positions, seq_of_token, cu_tokens, slots, A_log, dt_bias, q_scale, rows, gates, T, H, G, Dk, Dv);
+    const int widest = Dk > Dv ? Dk : Dv;
+    if (Dk % 4 == 0 && Dv % 4 == 0 && widest <= 256 && K <= 4 && ld % 4 == 0 && state_stride % 4 == 0 && kept % 4 == 0 &&
+        ((uintptr_t)proj | (uintptr_t)rows | (uintptr_t)state) % 16 == 0) {
+        const long long warps = (long long)((T + RUN - 1) / RUN) * (2 * G + H + 1);
+        const dim3 grid((unsigned)((warps + PREP_THREADS / 32 - 1) / (PREP_THREADS / 32)));
+#define DR_PREP(K_, NQ_)                                                                                                                                      \
+    vm_launch_pdl(delta_prepare_run_kernel<K_, NQ_>, grid, dim3(PREP_THREADS), 0, stream, proj, ld, b_off, a_off, taps, (const float*)state, state_stride, kept, \
+                  positions, seq_of_token, cu_tokens, slots, A_log, dt_bias, q_scale, rows, gates, T, H, G, Dk, Dv)
+#define DR_PREP_K(NQ_)                   \
+    do {                                 \
+        if (K == 1) DR_PREP(1, NQ_);     \
+        else if (K == 2) DR_PREP(2, NQ_); \
+        else if (K == 3) DR_PREP(3, NQ_); \
+        else DR_PREP(4, NQ_);            \
+    } while (0)
+        if (widest <= 128) DR_PREP_K(1);
+        else DR_PREP_K(2);
+#undef DR_PREP_K
+#undef DR_PREP
+    } else {
+        const cudaError_t e = allow_smem(delta_prepare_kernel, smem);
+        if (e != cudaSuccess) return (int)e;
+        vm_launch_pdl(delta_prepare_kernel, dim3((T + PT - 1) / PT, 2 * G + H + 1), dim3(PREP_THREADS), smem, stream, proj, ld, b_off, a_off, taps, K,
+                      (const float*)state, state_stride, kept, positions, seq_of_token, cu_tokens, slots, A_log, dt_bias, q_scale, rows, gates, T, H, G, Dk, Dv);
+    }
     const int st = vm_launch_status();
     if (st || K <= 1) return st;
     const int slices = (C + 255) / 256;

@@ -126,6 +126,80 @@ __global__ void mixer_prepare_kernel(const float* __restrict__ proj, int ld, con
         }
 }
 
+// The preparation without convolution, norm over the projection and rotation: bias, heads divided by their root mean square (or not), q out, k
+// and v to the cache page.  A warp per head of a token, two neighbouring values per lane and turn; nothing passes through shared memory.
+constexpr int HEADS_THREADS = 256;
+__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+
+template <typename T, int NP>               // NP: pairs of values a lane keeps (heads of up to 64 NP values)
+__global__ void __launch_bounds__(HEADS_THREADS)
+mixer_heads_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias, float eps, const int* __restrict__ positions,
+                   const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int max_blocks, T* __restrict__ q_out,
+                   T* __restrict__ kpages, T* __restrict__ vpages, int n_pages, int n_tokens, int H, int G, int Dk, int Dv, int unit_heads,
+                   int* __restrict__ err) {
+    vm_pdl_launch_dependents();
+    const int items = H + 2 * G, lane = threadIdx.x & 31;
+    const long long w = (long long)blockIdx.x * (HEADS_THREADS / 32) + (threadIdx.x >> 5);
+    const int t = (int)(w / items), item = (int)(w - (long long)t * items);
+    if (t >= n_tokens) return;
+    const bool is_v = item >= H + G;
+    const int D = is_v ? Dv : Dk, col = is_v ? (H + G) * Dk + (item - H - G) * Dv : item * Dk;
+    float2 b[NP];
+#pragma unroll
+    for (int n = 0; n < NP; ++n) {
+        const int d = 2 * (lane + 32 * n);
+        b[n] = bias && d < D ? *reinterpret_cast<const float2*>(bias + col + d) : make_float2(0.f, 0.f);
+    }
+    vm_pdl_wait();
+    float2 x[NP];
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NP; ++n) {
+        const int d = 2 * (lane + 32 * n);
+        x[n] = d < D ? *reinterpret_cast<const float2*>(proj + (size_t)t * ld + col + d) : make_float2(0.f, 0.f);
+        x[n].x += b[n].x;
+        x[n].y += b[n].y;
+        ss += x[n].x * x[n].x + x[n].y * x[n].y;
+    }
+    T* dst;
+    if (item < H) {
+        dst = q_out + (size_t)t * H * Dk + (size_t)item * Dk;
+    } else {
+        const int pos = positions[t], blk = pos / VM_PAGE_TOKENS;
+        const int page = blk < max_blocks ? block_table[(size_t)seq_of_token[t] * max_blocks + blk] : -1;
+        if (page < 0 || page >= n_pages) {
+            if (lane == 0 && err) atomicExch(err, VM_ERRWORD_CACHE_WRITE);
+            return;
+        }
+        const int g = is_v ? item - H - G : item - H;
+        dst = (is_v ? vpages : kpages) + (((size_t)page * G + g) * VM_PAGE_TOKENS + pos % VM_PAGE_TOKENS) * D;
+    }
+    const float f = unit_heads && !is_v ? 1.0f / sqrtf(vm_warp_sum(ss) / (float)D + eps) : 1.0f;
+#pragma unroll
+    for (int n = 0; n < NP; ++n) {
+        const int d = 2 * (lane + 32 * n);
+        if (d < D) store2(dst + d, x[n].x * f, x[n].y * f);
+    }
+}
+
+template <typename T>
+static int launch_heads(const float* proj, int ld, const float* bias, float eps, const int* positions, const int* seq_of_token, const int* block_table,
+                        int max_blocks, T* q_out, T* kpages, T* vpages, int n_pages, int n_tokens, int H, int G, int Dk, int Dv, int unit_heads, int* err,
+                        cudaStream_t stream) {
+    const long long warps = (long long)n_tokens * (H + 2 * G);
+    const dim3 grid((unsigned)((warps + HEADS_THREADS / 32 - 1) / (HEADS_THREADS / 32)));
+    const int widest = Dk > Dv ? Dk : Dv;
+#define VM_HEADS(NP_)                                                                                                                                 \
+    vm_launch_pdl(mixer_heads_kernel<T, NP_>, grid, dim3(HEADS_THREADS), 0, stream, proj, ld, bias, eps, positions, seq_of_token, block_table, max_blocks, \
+                  q_out, kpages, vpages, n_pages, n_tokens, H, G, Dk, Dv, unit_heads, err)
+    if (widest <= 64) VM_HEADS(1);
+    else if (widest <= 128) VM_HEADS(2);
+    else VM_HEADS(4);
+#undef VM_HEADS
+    return vm_launch_status();
+}
+
 // the kept rows of every sequence move on by the step's tokens: row K - 1 - d holds the projected row d places before the next step
 __global__ void mixer_keep_rows_kernel(const float* __restrict__ proj, int ld, int C, int K, float* __restrict__ state, long long state_stride,
                                        int state_offset, const int* __restrict__ cu_tokens, const int* __restrict__ slots) {
@@ -161,6 +235,15 @@ VM_API int vm_mixer_prepare(const float* proj, int ld, const float* bias, const 
     if ((q_norm != nullptr) != (k_norm != nullptr)) return VM_ERR_BAD_ARG;
     if (inv_freq && (rotary_dim < 0 || rotary_dim > Dk || rotary_dim % 2)) return VM_ERR_BAD_ARG;
     if (!taps) K = 0;
+    if (!taps && !q_norm && !inv_freq && !values_are_keys && (G == 0 || kpages) && Dk % 2 == 0 && Dv % 2 == 0 && ld % 2 == 0 && Dk <= 256 && Dv <= 256 &&
+        ((uintptr_t)proj | (uintptr_t)bias) % 8 == 0) {
+        if (act_dtype == VM_F32)
+            return launch_heads<float>(proj, ld, bias, eps, positions, seq_of_token, block_table, max_blocks, (float*)q_out, (float*)kpages, (float*)vpages, n_pages,
+                                       T, H, G, Dk, Dv, unit_heads, err, stream);
+        if (act_dtype == VM_BF16)
+            return launch_heads<__nv_bfloat16>(proj, ld, bias, eps, positions, seq_of_token, block_table, max_blocks, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kpages,
+                                               (__nv_bfloat16*)vpages, n_pages, T, H, G, Dk, Dv, unit_heads, err, stream);
+    }
     const int C = (H + G) * Dk + (values_are_keys ? 0 : G * Dv);
     const size_t smem = (size_t)C * sizeof(float);
     if (smem > 160 * 1024) return VM_ERR_UNSUPPORTED;
@@ -201,11 +284,36 @@ __global__ void sigmoid_gate_heads_kernel(T* __restrict__ x, const float* __rest
     }
 }
 
+// bfloat16 with heads of a multiple of eight values: eight values and one gate per thread
+__global__ void __launch_bounds__(256)
+sigmoid_gate_heads_vec_kernel(__nv_bfloat16* __restrict__ x, const float* __restrict__ g, int ldg, int cols, int per, long long n_vec) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const int per_row = cols >> 3;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n_vec; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / per_row;
+        const int c = (int)(i - t * per_row) << 3;
+        uint4* px = reinterpret_cast<uint4*>(x + t * cols + c);
+        uint4 d = *px;
+        const float f = 1.0f / (1.0f + expf(-g[t * ldg + c / per]));
+        __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&d);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[k] = __floats2bfloat162_rn(__low2float(v[k]) * f, __high2float(v[k]) * f);
+        *px = d;
+    }
+}
+
 VM_API int vm_sigmoid_gate_heads(void* x, const float* g, int ldg, int T, int cols, int per, int act_dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (cols <= 0 || per <= 0) return VM_ERR_BAD_ARG;
     const long long n = (long long)T * cols, want = (n + 255) / 256;
     const int grid = (int)(want < 148 * 16 ? want : 148 * 16);
+    if (act_dtype == VM_BF16 && per % 8 == 0 && cols % 8 == 0 && (uintptr_t)x % 16 == 0) {
+        const long long n_vec = n / 8, want_vec = (n_vec + 255) / 256;
+        vm_launch_pdl(sigmoid_gate_heads_vec_kernel, dim3((unsigned)(want_vec < 148 * 16 ? want_vec : 148 * 16)), dim3(256), 0, stream, (__nv_bfloat16*)x, g, ldg,
+                      cols, per, n_vec);
+        return vm_launch_status();
+    }
     if (act_dtype == VM_F32) vm_launch_pdl(sigmoid_gate_heads_kernel<float>, dim3(grid), dim3(256), 0, stream, (float*)x, g, ldg, cols, per, n);
     else if (act_dtype == VM_BF16) vm_launch_pdl(sigmoid_gate_heads_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, (__nv_bfloat16*)x, g, ldg, cols, per, n);
     else return VM_ERR_UNSUPPORTED;
