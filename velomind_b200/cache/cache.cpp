@@ -66,8 +66,9 @@ PageBook::PageBook(const CacheNeed& need_, int n_pages_, int max_slots_, int max
     : need(need_), n_pages(n_pages_), max_slots(max_slots_), max_blocks(max_blocks_), pages(n_pages_, "cache page"),
       blocks_begin(static_cast<size_t>(max_slots_), 0), blocks_end(static_cast<size_t>(max_slots_), 0),
       table_(static_cast<size_t>(max_slots_) * max_blocks_, -1) {
-    if (need.kind != CacheNeed::All && need.kind != CacheNeed::Window) throw CacheError("a cache group holds keys and values; a need of kind 'none' has none");
+    if (need.kind == CacheNeed::None) throw CacheError("a cache group holds keys and values; a need of kind 'none' has none");
     if (need.kind == CacheNeed::Window && need.window <= 0) throw CacheError("a window group needs window > 0");
+    if (need.kind == CacheNeed::Chunk && need.chunk <= 0) throw CacheError("a chunk group needs chunk > 0");
     if (need.key_dim <= 0 || need.value_dim < 0)                    // value_dim 0: one row per token and no second one (a latent that serves as both)
         throw CacheError(format("a cache group stores keys of a positive size and values of a size >= 0; a mixer asked for %d and %d", need.key_dim,
                                 need.value_dim));
@@ -90,10 +91,10 @@ void PageBook::ensure(int slot, int new_len) {
 }
 
 void PageBook::trim(int slot, int length) {
-    if (need.kind != CacheNeed::Window) return;
+    if (need.kind != CacheNeed::Window && need.kind != CacheNeed::Chunk) return;
     // the next query sits at position `length` or later and sees keys at positions > length - window
-    // (the blocks of the first keep_first tokens stay: every later query sees them)
-    const int first_needed = std::max(0, length - need.window + 1);
+    // (the blocks of the first keep_first tokens stay: every later query sees them); in a chunk group it sees its own chunk's keys
+    const int first_needed = need.kind == CacheNeed::Chunk ? length - length % need.chunk : std::max(0, length - need.window + 1);
     int b = std::max(blocks_begin[slot], std::min(kept_blocks(), blocks_end[slot]));
     while (b < blocks_end[slot] && (b + 1) * VM_PAGE_TOKENS <= first_needed) {
         int& entry = table_[static_cast<size_t>(slot) * max_blocks + b];

@@ -367,7 +367,9 @@ const char* vmb_engine_stats(void* e) {
         json::Array groups;
         for (size_t g = 0; g < book.groups.size(); ++g) {
             json::Value o;
-            o.set("kind", book.groups[g].need.kind == CacheNeed::Window ? "window" : "all");
+            const CacheNeed::Kind kind = book.groups[g].need.kind;
+            o.set("kind", kind == CacheNeed::Window ? "window" : (kind == CacheNeed::Chunk ? "chunk" : "all"));
+            o.set("chunk", book.groups[g].need.chunk);
             o.set("window", book.groups[g].need.window);
             o.set("layers", book.layers_in_group[g]);
             o.set("pages_held", book.groups[g].pages.held_count());

@@ -6,6 +6,7 @@
 //   score(i, j) = scale q_i . k_j + rel[bucket(i - j), h]             bucket: a table from the distance to a row of `rel`
 //                                 - slope[h] (i - j)                  optional: a bias linear in the distance, one slope per head
 //   i sees j  iff  j <= i and (i - j < window  or  j < keep_first)    window 0: every earlier key
+//                  with a chunked mask also j >= chunk floor(i / chunk): keys of the query's own chunk of places (kept ones stay)
 //   out_i = softmax_j(score) v_j
 //
 // Keys have `Dk` values per head and values `Dv`; the paged cache keeps them in pools of their own
@@ -79,7 +80,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
                                    const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                                    const int* __restrict__ seq_of_token, const float* __restrict__ rel, const int* __restrict__ bucket_of, int far,
                                    T* __restrict__ out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
-                                   int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes, int v_stride, int* __restrict__ err) {
+                                   int chunk, int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes, int v_stride, int* __restrict__ err) {
     extern __shared__ float qs_all[];                       // ATT_WARPS x Dk
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long w = (long long)blockIdx.x * ATT_WARPS + warp;
@@ -92,7 +93,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
     for (int d = lane; d < Dk; d += 32) qs[d] = vm_to_float(qrow[d]) * scale;
     __syncwarp();
 
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;      // the window is [lo, pos]
+    const int lo = vm_first_seen(pos, window, chunk);                                 // the window is [lo, pos]
     const int kept = min(keep_first, lo);                                             // keys [0, kept) are seen although outside it
     const int first_window_chunk = (lo / 32) * 32;
     const float slope = slopes ? slopes[h] : 0.f;
@@ -159,7 +160,7 @@ __global__ void attn_biased_kernel(const T* __restrict__ q, int q_row_stride, co
 template <typename T>
 int launch_biased(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                   const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, void* out, int n_tokens, int H,
-                  int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, const float* sink, const float* slopes, int v_stride, int* err,
+                  int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int chunk, int n_pages, const float* sink, const float* slopes, int v_stride, int* err,
                   cudaStream_t stream) {
     const long long warps = (long long)n_tokens * H;
     const int blocks = (int)((warps + ATT_WARPS - 1) / ATT_WARPS);
@@ -171,7 +172,7 @@ int launch_biased(const void* q, int q_row_stride, const void* kpages, const voi
         attn_biased_kernel<T, E><<<blocks, ATT_WARPS * 32, smem, stream>>>((const T*)q, q_row_stride, (const T*)kpages, (const T*)vpages, \
                                                                            block_table, max_blocks, positions, seq_of_token, rel,       \
                                                                            bucket_of, far, (T*)out, n_tokens, H, Hkv, Dk, Dv, scale,     \
-                                                                           window, keep_first, n_pages, sink, slopes, v_stride, err);    \
+                                                                           window, keep_first, chunk, n_pages, sink, slopes, v_stride, err);    \
         break;
     switch (epl) {
         VM_ATT_CASE(1) VM_ATT_CASE(2) VM_ATT_CASE(3) VM_ATT_CASE(4) VM_ATT_CASE(5) VM_ATT_CASE(6) VM_ATT_CASE(7) VM_ATT_CASE(8)
@@ -212,27 +213,27 @@ VM_API int vm_attention_biased_generic(const void* q, int q_row_stride, const vo
                                        int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages,
                                        int act_dtype, int* err, cudaStream_t stream) {
     return vm_attention_sink_generic(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, nullptr, nullptr, 0, out,
-                                     n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, act_dtype, err, stream);
+                                     n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, 0, n_pages, act_dtype, err, stream);
 }
 
 // The same with a sink and values that may lie inside the key rows.  sink float32 [H] (null: none): exp(sink[h]) is one more term
 // of head h's softmax denominator, without a key or a value, not scaled.  v_row_stride: elements from one token's value row to the
 // next in `vpages` (0: Dv); with vpages == kpages and v_row_stride == Dk a token's value is the first Dv values of its key row.
-// slopes float32 [H] (null: none): slopes[h] * (i - j) is taken off head h's score of key j.
+// slopes float32 [H] (null: none): slopes[h] * (i - j) is taken off head h's score of key j.  chunk > 0: a chunked mask.
 VM_API int vm_attention_sink_generic(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                                      const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, const float* sink,
                                      const float* slopes, int v_row_stride, void* out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
-                                     int n_pages, int act_dtype, int* err, cudaStream_t stream) {
+                                     int chunk, int n_pages, int act_dtype, int* err, cudaStream_t stream) {
     const int v_stride = v_row_stride > 0 ? v_row_stride : Dv;
     if (v_stride < Dv) return VM_ERR_BAD_ARG;
     if (n_tokens <= 0) return 0;
-    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dk > 2048 || Dv <= 0 || Dv > 1024 || window < 0 || keep_first < 0) return VM_ERR_UNSUPPORTED;
+    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dk > 2048 || Dv <= 0 || Dv > 1024 || window < 0 || keep_first < 0 || chunk < 0) return VM_ERR_UNSUPPORTED;
     if ((rel != nullptr) != (bucket_of != nullptr) || (rel && far < 0)) return VM_ERR_BAD_ARG;
     if (act_dtype == VM_F32)
         return launch_biased<float>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, out, n_tokens, H,
-                                    Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err, stream);
+                                    Hkv, Dk, Dv, scale, window, keep_first, chunk, n_pages, sink, slopes, v_stride, err, stream);
     if (act_dtype == VM_BF16)
         return launch_biased<__nv_bfloat16>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, seq_of_token, rel, bucket_of, far, out,
-                                            n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err, stream);
+                                            n_tokens, H, Hkv, Dk, Dv, scale, window, keep_first, chunk, n_pages, sink, slopes, v_stride, err, stream);
     return VM_ERR_UNSUPPORTED;
 }

@@ -1,7 +1,8 @@
 // The bfloat16 kernels of the windowed attention with a distance bias and kept first tokens (arithmetic and arguments as in
 // attention_biased.cu): prompts on the tensor cores, decode steps with the keys of one query dealt out to the warps of a CTA.
 //
-// Both take, beside or instead of the table, a bias linear in the distance: slope[h] (i - j) comes off head h's score.
+// Both take, beside or instead of the table, a bias linear in the distance: slope[h] (i - j) comes off head h's score; and a chunked
+// mask: only keys of the query's own chunk of places (and kept ones) are seen.
 //
 // Prompts.  One CTA owns 64 consecutive new tokens of one sequence and one query head; its four warps own 16 query rows
 // each.  The key blocks a tile can see are the pages of the kept first tokens and the pages its rows' windows touch; they
@@ -41,7 +42,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
                            const __nv_bfloat16* __restrict__ vpages, const int* __restrict__ block_table, int max_blocks,
                            const int* __restrict__ positions, const int* __restrict__ cu_tokens, int B, const float* __restrict__ rel,
                            const int* __restrict__ bucket_of, int far, int rel_rows, __nv_bfloat16* __restrict__ out, int H, int Hkv,
-                           float scale_log2, int window, int keep_first, int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes,
+                           float scale_log2, int window, int keep_first, int chunk, int n_pages, const float* __restrict__ sink, const float* __restrict__ slopes,
                            int* __restrict__ err) {
     constexpr int KP = DK + 8, VP = VK ? KP : DV + 8;     // padded rows: an odd number of 16-byte units -> no ldmatrix conflicts
     constexpr int KCH = DK / 8, VCH = DV / 8;   // 16-byte chunks per row
@@ -68,7 +69,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int pos0 = positions[t0];
     const int hi = pos0 + n_rows - 1;
-    const int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;      // the first row's window start: the tile's lowest
+    const int lo = vm_first_seen(pos0, window, chunk);      // the first row's window start: the tile's lowest
     const int blk_lo = lo / BN, blk_hi = hi / BN;
     // pages of kept first tokens that lie before the window's pages (keys below keep_first are seen by every row)
     const int kept_blocks = min((min(keep_first, lo) + BN - 1) / BN, blk_lo);
@@ -111,7 +112,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
     const int g = lane >> 2, t4 = lane & 3;
     const int row_a = warp * 16 + g, row_b = row_a + 8;
     const int pos_a = pos0 + row_a, pos_b = pos0 + row_b;
-    const int lo_a = (window > 0) ? pos_a - window + 1 : 0, lo_b = (window > 0) ? pos_b - window + 1 : 0;
+    const int lo_a = vm_first_seen(pos_a, window, chunk), lo_b = vm_first_seen(pos_b, window, chunk);
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
     float o[DV / 8][4];
 #pragma unroll
@@ -119,6 +120,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
     unsigned qa[DK / 16][4];
     bool q_loaded = false;
     const int warp_min_pos = pos0 + warp * 16, warp_max_pos = warp_min_pos + 15;
+    const int warp_lo = vm_first_seen(warp_min_pos, window, chunk);
     const float slope_log2 = sloped ? slopes[h] * LOG2E : 0.f;
 
     for (int step = 0; step < n_steps; ++step) {
@@ -136,8 +138,8 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
             q_loaded = true;
         }
         const int key0 = blk * BN;
-        // does any row of this warp see any key of this page?  (its window reaches down to warp_min_pos - window + 1)
-        const bool in_reach = key0 <= warp_max_pos && (window <= 0 || key0 + BN - 1 >= warp_min_pos - window + 1 || key0 < keep_first);
+        // does any row of this warp see any key of this page?  (its first row reaches lowest)
+        const bool in_reach = key0 <= warp_max_pos && (key0 + BN - 1 >= warp_lo || key0 < keep_first);
         if (in_reach && warp * 16 < n_rows) {
             const __nv_bfloat16* ks = sK + (size_t)buf * BN * KP;
             const __nv_bfloat16* vs = VK ? ks : sV + (size_t)buf * BN * VP;
@@ -240,7 +242,7 @@ attn_biased_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride
 template <int DK, int DV, bool VK>
 int launch_biased_prefill(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                           const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel, const int* bucket_of, int far,
-                          int rel_rows, void* out, int H, int Hkv, float scale, int window, int keep_first, int n_pages, const float* sink, const float* slopes,
+                          int rel_rows, void* out, int H, int Hkv, float scale, int window, int keep_first, int chunk, int n_pages, const float* sink, const float* slopes,
                           int* err, cudaStream_t stream) {
     const int table = rel ? (far + 1 <= DIRECT_TABLE_MAX ? far + 1 : rel_rows) : 0;
     const size_t smem = (size_t)(BM + 2 * BN) * (DK + 8) * sizeof(__nv_bfloat16) + (VK ? 0 : (size_t)2 * BN * (DV + 8) * sizeof(__nv_bfloat16)) +
@@ -254,7 +256,7 @@ int launch_biased_prefill(const void* q, int q_row_stride, const void* kpages, c
     }
     attn_biased_prefill_kernel<DK, DV, VK><<<dim3(n_tiles, H), 128, smem, stream>>>(
         (const __nv_bfloat16*)q, q_row_stride, (const __nv_bfloat16*)kpages, (const __nv_bfloat16*)vpages, block_table, max_blocks, positions,
-        cu_tokens, B, rel, bucket_of, far, rel_rows, (__nv_bfloat16*)out, H, Hkv, scale * 1.4426950408889634f, window, keep_first, n_pages, sink,
+        cu_tokens, B, rel, bucket_of, far, rel_rows, (__nv_bfloat16*)out, H, Hkv, scale * 1.4426950408889634f, window, keep_first, chunk, n_pages, sink,
         slopes, err);
     return vm_launch_status();
 }
@@ -268,7 +270,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32)
 attn_biased_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const __nv_bfloat16* __restrict__ kpages,
                           const __nv_bfloat16* __restrict__ vpages, const int* __restrict__ block_table, int max_blocks,
                           const int* __restrict__ positions, const float* __restrict__ rel, const int* __restrict__ bucket_of, int far,
-                          __nv_bfloat16* __restrict__ out, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages,
+                          __nv_bfloat16* __restrict__ out, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int chunk, int n_pages,
                           const float* __restrict__ sink, const float* __restrict__ slopes, int v_stride, int* __restrict__ err) {
     extern __shared__ __align__(16) float dsm[];            // [Dk] the query; then per warp: m, l, acc[Dv]
     float* qs = dsm;
@@ -281,7 +283,7 @@ attn_biased_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride,
     const __nv_bfloat16* qrow = q + (size_t)seq * q_row_stride + (size_t)h * Dk;
     for (int d = threadIdx.x; d < Dk; d += blockDim.x) qs[d] = __bfloat162float(qrow[d]) * scale;
     __syncthreads();
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = vm_first_seen(pos, window, chunk);
     const int kept = min(keep_first, lo);
     // the chunks of 32 keys (at absolute multiples of 32) that hold a visible key: those of the kept tokens, then those of the window
     const int kept_chunks = min((kept + 31) / 32, lo / 32);
@@ -417,25 +419,25 @@ VM_API int vm_attention_biased_prefill_bf16(const void* q, int q_row_stride, con
                                             const int* bucket_of, int far, int rel_rows, void* out, int H, int Hkv, int Dk, int Dv, float scale,
                                             int window, int keep_first, int n_pages, int* err, cudaStream_t stream) {
     return vm_attention_sink_prefill_bf16(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, cu_tokens, B, n_tiles, rel, bucket_of, far,
-                                          rel_rows, nullptr, nullptr, 0, out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, err, stream);
+                                          rel_rows, nullptr, nullptr, 0, out, H, Hkv, Dk, Dv, scale, window, keep_first, 0, n_pages, err, stream);
 }
 
 // The same with a sink (float32 [H], null: none; exp(sink[h]) joins head h's denominator), slopes (float32 [H], null: none; slopes[h] (i - j)
-// comes off the score) and, with vpages == kpages and
+// comes off the score), a chunked mask (chunk > 0) and, with vpages == kpages and
 // v_row_stride == Dk, values that are the first Dv values of the key rows (sizes: vm_attention_sink_prefill_fits).
 VM_API int vm_attention_sink_prefill_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table,
                                           int max_blocks, const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel,
                                           const int* bucket_of, int far, int rel_rows, const float* sink, const float* slopes, int v_row_stride, void* out, int H, int Hkv,
-                                          int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err, cudaStream_t stream) {
+                                          int Dk, int Dv, float scale, int window, int keep_first, int chunk, int n_pages, int* err, cudaStream_t stream) {
     if (n_tiles <= 0 || B <= 0) return 0;
-    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || (q_row_stride % 8) != 0 || window < 0 || keep_first < 0) return VM_ERR_UNSUPPORTED;
+    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || (q_row_stride % 8) != 0 || window < 0 || keep_first < 0 || chunk < 0) return VM_ERR_UNSUPPORTED;
     if ((rel != nullptr) != (bucket_of != nullptr) || (rel && (far < 0 || rel_rows <= 0))) return VM_ERR_BAD_ARG;
     const bool in_keys = vpages == kpages && v_row_stride == Dk && Dv < Dk;
     if (!in_keys && v_row_stride != 0 && v_row_stride != Dv) return VM_ERR_UNSUPPORTED;
 #define VM_BP(K, V, IN)                                                                                                                        \
     if (Dk == K && Dv == V && in_keys == IN)                                                                                                   \
         return launch_biased_prefill<K, V, IN>(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, cu_tokens, B, n_tiles, rel, \
-                                               bucket_of, far, rel_rows, out, H, Hkv, scale, window, keep_first, n_pages, sink, slopes, err, stream);
+                                               bucket_of, far, rel_rows, out, H, Hkv, scale, window, keep_first, chunk, n_pages, sink, slopes, err, stream);
     VM_BP(32, 16, false) VM_BP(32, 32, false) VM_BP(32, 64, false) VM_BP(32, 128, false)
     VM_BP(64, 16, false) VM_BP(64, 32, false) VM_BP(64, 64, false) VM_BP(64, 128, false)
     VM_BP(96, 16, false) VM_BP(96, 32, false) VM_BP(96, 64, false) VM_BP(96, 128, false)
@@ -454,16 +456,16 @@ VM_API int vm_attention_biased_decode_bf16(const void* q, int q_row_stride, cons
                                            int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err,
                                            cudaStream_t stream) {
     return vm_attention_sink_decode_bf16(q, q_row_stride, kpages, vpages, block_table, max_blocks, positions, rel, bucket_of, far, nullptr, nullptr, 0, out, B, H, Hkv,
-                                         Dk, Dv, scale, window, keep_first, n_pages, err, stream);
+                                         Dk, Dv, scale, window, keep_first, 0, n_pages, err, stream);
 }
 
 // the same with a sink, slopes and a stride between value rows (0: Dv), as vm_attention_sink_generic
 VM_API int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table,
                                          int max_blocks, const int* positions, const float* rel, const int* bucket_of, int far, const float* sink,
                                          const float* slopes, int v_row_stride, void* out, int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
-                                         int n_pages, int* err, cudaStream_t stream) {
+                                         int chunk, int n_pages, int* err, cudaStream_t stream) {
     if (B <= 0) return 0;
-    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dk > 1024 || Dv <= 0 || Dv > 256 || window < 0 || keep_first < 0) return VM_ERR_UNSUPPORTED;
+    if (H <= 0 || Hkv <= 0 || H % Hkv != 0 || Dk <= 0 || Dk > 1024 || Dv <= 0 || Dv > 256 || window < 0 || keep_first < 0 || chunk < 0) return VM_ERR_UNSUPPORTED;
     if ((rel != nullptr) != (bucket_of != nullptr) || (rel && far < 0)) return VM_ERR_BAD_ARG;
     if (H > 65535) return VM_ERR_UNSUPPORTED;
     const int v_stride = v_row_stride > 0 ? v_row_stride : Dv;
@@ -475,7 +477,7 @@ VM_API int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const 
     case V:                                                                                                                                   \
         e = vm_launch_pdl(attn_biased_decode_kernel<V>, grid, dim3(DEC_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, q_row_stride,      \
                           (const __nv_bfloat16*)kpages, (const __nv_bfloat16*)vpages, block_table, max_blocks, positions, rel, bucket_of, far, \
-                          (__nv_bfloat16*)out, H, Hkv, Dk, Dv, scale, window, keep_first, n_pages, sink, slopes, v_stride, err);               \
+                          (__nv_bfloat16*)out, H, Hkv, Dk, Dv, scale, window, keep_first, chunk, n_pages, sink, slopes, v_stride, err);               \
         break;
     switch ((Dv + 63) / 64) {
         VM_BD(1) VM_BD(2) VM_BD(3) VM_BD(4)

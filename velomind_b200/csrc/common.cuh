@@ -39,6 +39,14 @@ __device__ __forceinline__ float vm_block_sum(float v, float* red) {
     return vm_warp_sum(t);
 }
 
+// The first key a query at place `pos` sees: a window reaches window - 1 places back (0: to the start), a chunked mask to the start of the
+// query's chunk of `chunk` places (chunks are counted from the sequence's start; 0: none).
+__device__ __forceinline__ int vm_first_seen(int pos, int window, int chunk) {
+    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (chunk > 0) lo = max(lo, pos - pos % chunk);
+    return lo;
+}
+
 // ---- programmatic dependent launch: a kernel launched through vm_launch_pdl may begin (and fetch data that
 // no earlier kernel writes, i.e. weights) while its predecessor in the stream is still running; it must call
 // vm_pdl_wait() before it reads anything an earlier kernel wrote and before its first global write.

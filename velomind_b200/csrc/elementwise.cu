@@ -273,6 +273,53 @@ __global__ void gated_activation_kernel(const T* __restrict__ gu, T* __restrict_
     }
 }
 
+// the clamped unit: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1)
+template <typename T>
+__global__ void clamped_unit_kernel(const T* __restrict__ gu, T* __restrict__ out, int T_, int I, float limit, float alpha) {
+    const size_t n = (size_t)T_ * I;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = idx / I;
+        const int i = (int)(idx - t * I);
+        const float g = fminf(vm_to_float(gu[t * 2 * I + i]), limit), u = fminf(fmaxf(vm_to_float(gu[t * 2 * I + I + i]), -limit), limit);
+        out[idx] = vm_from_float<T>(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+    }
+}
+
+// bfloat16, I % 8 == 0: eight values per load and store (float32 throughout, as in the SiLU unit above)
+__global__ void clamped_unit_bf16_vec_kernel(const uint4* __restrict__ gu, uint4* __restrict__ out, size_t n8, int I8, float limit, float alpha) {
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n8; idx += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = idx / I8;
+        const int i = (int)(idx - t * I8);
+        const uint4 g4 = gu[t * 2 * I8 + i], u4 = gu[t * 2 * I8 + I8 + i];
+        const unsigned gw[4] = {g4.x, g4.y, g4.z, g4.w}, uw[4] = {u4.x, u4.y, u4.z, u4.w};
+        unsigned ow[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[k]));
+            const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[k]));
+            const float ga = fminf(g.x, limit), gb = fminf(g.y, limit);
+            const float ua = fminf(fmaxf(u.x, -limit), limit) + 1.0f, ub = fminf(fmaxf(u.y, -limit), limit) + 1.0f;
+            const __nv_bfloat162 o2 = __floats2bfloat162_rn(ga * __frcp_rn(1.0f + __expf(-alpha * ga)) * ua, gb * __frcp_rn(1.0f + __expf(-alpha * gb)) * ub);
+            ow[k] = *reinterpret_cast<const unsigned*>(&o2);
+        }
+        out[idx] = make_uint4(ow[0], ow[1], ow[2], ow[3]);
+    }
+}
+
+// the clamped gated unit: out[t, i] from gate_up[t, i] and gate_up[t, I + i]
+VM_API int vm_clamped_unit(const void* gate_up, void* out, int T, int I, float limit, float alpha, int act_dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (I <= 0 || !(limit > 0.f)) return VM_ERR_BAD_ARG;
+    const bool vec = act_dtype == VM_BF16 && I % 8 == 0 && ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const size_t n = (size_t)T * (vec ? I / 8 : I), want = (n + 255) / 256;
+    const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+    if (vec) clamped_unit_bf16_vec_kernel<<<blocks, 256, 0, stream>>>((const uint4*)gate_up, (uint4*)out, n, I / 8, limit, alpha);
+    else if (act_dtype == VM_F32) clamped_unit_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gate_up, (float*)out, T, I, limit, alpha);
+    else if (act_dtype == VM_BF16) clamped_unit_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, T, I, limit, alpha);
+    else return VM_ERR_UNSUPPORTED;
+    return vm_launch_status();
+}
+
 VM_API int vm_gated_activation(const void* gate_up, void* out, int T, int I, int kind, int act_dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (kind == VM_ACT_SILU) return vm_swiglu(gate_up, out, T, I, act_dtype, stream);

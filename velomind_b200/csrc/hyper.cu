@@ -212,7 +212,7 @@ template <typename W>
 __global__ void embed_pairs_kernel(const W* __restrict__ table, const W* __restrict__ pairs, const int* __restrict__ tokens,
                                    const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ cu_tokens,
                                    const int* __restrict__ slots, int* __restrict__ last, long long last_stride, int keep_here, float* __restrict__ out,
-                                   int hid, int vocab, long long buckets, long long mul_prev, long long mul_cur, int* __restrict__ err) {
+                                   int hid, int vocab, long long buckets, long long mul_prev, long long mul_cur, float scale, int* __restrict__ err) {
     vm_pdl_launch_dependents();
     vm_pdl_wait();
     const int t = blockIdx.x;
@@ -227,7 +227,7 @@ __global__ void embed_pairs_kernel(const W* __restrict__ table, const W* __restr
     }
     const W* a = table + (size_t)(ok ? id : 0) * hid;
     const W* b = pairs + (size_t)row * hid;
-    for (int i = threadIdx.x; i < hid; i += blockDim.x) out[(size_t)t * hid + i] = ok ? vm_to_float(a[i]) + vm_to_float(b[i]) : 0.f;
+    for (int i = threadIdx.x; i < hid; i += blockDim.x) out[(size_t)t * hid + i] = ok ? fmaf(vm_to_float(a[i]), scale, vm_to_float(b[i])) : 0.f;
     if (keep_here) {                         // one token per sequence: this block alone reads and writes the sequence's word
         __syncthreads();
         if (threadIdx.x == 0) last[(size_t)slots[seq] * last_stride] = id;
@@ -242,20 +242,20 @@ __global__ void embed_pairs_keep_kernel(const int* __restrict__ tokens, const in
     if (b < B && cu_tokens[b + 1] > cu_tokens[b]) last[(size_t)slots[b] * last_stride] = tokens[cu_tokens[b + 1] - 1];
 }
 
-// table [vocab, hid] and pairs [buckets + 1, hid] in one dtype; `last`: an int32 word per slot, last_stride words apart
+// table [vocab, hid] (its rows times `scale`) and pairs [buckets + 1, hid] in one dtype; `last`: an int32 word per slot, last_stride words apart
 VM_API int vm_embed_pairs(const void* table, const void* pairs, int table_dtype, const int* tokens, const int* positions, const int* seq_of_token,
                           const int* cu_tokens, const int* slots, int* last, long long last_stride, float* out, int T, int B, int hid, int vocab,
-                          long long buckets, long long mul_prev, long long mul_cur, int one_token_each, int* err, cudaStream_t stream) {
+                          long long buckets, long long mul_prev, long long mul_cur, float scale, int one_token_each, int* err, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (buckets <= 0 || !last) return VM_ERR_BAD_ARG;
     const int threads = hid >= 512 ? 256 : 128;
     if (table_dtype == VM_F32)
         vm_launch_pdl(embed_pairs_kernel<float>, dim3(T), dim3(threads), 0, stream, (const float*)table, (const float*)pairs, tokens, positions,
-                      seq_of_token, cu_tokens, slots, last, last_stride, one_token_each, out, hid, vocab, buckets, mul_prev, mul_cur, err);
+                      seq_of_token, cu_tokens, slots, last, last_stride, one_token_each, out, hid, vocab, buckets, mul_prev, mul_cur, scale, err);
     else if (table_dtype == VM_BF16)
         vm_launch_pdl(embed_pairs_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (const __nv_bfloat16*)table, (const __nv_bfloat16*)pairs,
                       tokens, positions, seq_of_token, cu_tokens, slots, last, last_stride, one_token_each, out, hid, vocab, buckets, mul_prev, mul_cur,
-                      err);
+                      scale, err);
     else return VM_ERR_UNSUPPORTED;
     int st = vm_launch_status();
     if (st || one_token_each) return st;

@@ -191,11 +191,11 @@ __global__ void router_kernel(const void* __restrict__ x, const float* __restric
 //   s = softmax(z) over all n_out outputs;  choice = s + correction (the correction steers the choice, not the weights)
 //   outputs form `group_count` equal groups of neighbours; a group's score is its largest choice score; only outputs of the
 //   `group_keep` best groups can be chosen (the lowest group index wins a tie, as the lowest output index does below)
-//   the `top` largest choice scores are chosen; weight = s * scale, not renormalised
+//   the `top` largest choice scores are chosen; weight = s * scale, not renormalised (`normalize`: s / (sum of the chosen s + 1e-20) * scale)
 template <typename T>
 __global__ void router_scored_kernel(const void* __restrict__ x, const float* __restrict__ norm_w, float eps, const float* __restrict__ w_router,
                                      const float* __restrict__ correction, int hidden, int n_out, int top, int group_count, int group_keep,
-                                     int group_top, float scale, int score_kind, int* __restrict__ chosen, float* __restrict__ weight) {
+                                     int group_top, float scale, int score_kind, int normalize, int* __restrict__ chosen, float* __restrict__ weight) {
     __shared__ float red[32];
     extern __shared__ __align__(16) float sm[];          // [hidden] input, [n_out] scores, [n_out] choice scores, [group_count] group scores
     float* xs = sm;
@@ -267,6 +267,7 @@ __global__ void router_scored_kernel(const void* __restrict__ x, const float* __
         }
         __syncwarp();
     }
+    float sum_chosen = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;
@@ -281,12 +282,17 @@ __global__ void router_scored_kernel(const void* __restrict__ x, const float* __
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (at == 0x7fffffff) at = 0;                      // fewer eligible outputs than `top` (a configuration the host refuses)
+        sum_chosen += sc[at];
         if (lane == 0) {
             chosen[(size_t)t * top + k] = at;
             weight[(size_t)t * top + k] = sc[at] * scale;
             ch[at] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (normalize) {
+        const float inv = scale / (sum_chosen + 1e-20f);
+        for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] = sc[chosen[(size_t)t * top + k]] * inv;
     }
 }
 
@@ -511,14 +517,14 @@ VM_API int vm_expert_router_scored(const void* x, const float* norm_w, float eps
 VM_API int vm_expert_router_scores(const void* x, const float* norm_w, float eps, const float* w_router, const float* correction, int T, int hidden,
                                    int n_out, int top, int group_count, int group_keep, float scale, int score_kind, int* chosen, float* weight,
                                    int act_dtype, cudaStream_t stream) {
-    return vm_expert_router_groups(x, norm_w, eps, w_router, correction, T, hidden, n_out, top, group_count, group_keep, 1, scale, score_kind, chosen,
+    return vm_expert_router_groups(x, norm_w, eps, w_router, correction, T, hidden, n_out, top, group_count, group_keep, 1, scale, score_kind, 0, chosen,
                                    weight, act_dtype, stream);
 }
 
 // the same with the number of a group's largest scores whose sum is the group's score
 VM_API int vm_expert_router_groups(const void* x, const float* norm_w, float eps, const float* w_router, const float* correction, int T, int hidden,
-                                   int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, int* chosen,
-                                   float* weight, int act_dtype, cudaStream_t stream) {
+                                   int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, int normalize,
+                                   int* chosen, float* weight, int act_dtype, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (group_top < 1) return VM_ERR_BAD_ARG;
     if (score_kind != VM_SCORE_SOFTMAX && score_kind != VM_SCORE_SIGMOID) return VM_ERR_BAD_ARG;
@@ -528,10 +534,10 @@ VM_API int vm_expert_router_groups(const void* x, const float* norm_w, float eps
     if (smem > 48 * 1024) return VM_ERR_UNSUPPORTED;
     if (act_dtype == VM_F32)
         vm_launch_pdl(router_scored_kernel<float>, dim3(T), dim3(256), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top, group_count,
-                      group_keep, group_top, scale, score_kind, chosen, weight);
+                      group_keep, group_top, scale, score_kind, normalize, chosen, weight);
     else if (act_dtype == VM_BF16)
         vm_launch_pdl(router_scored_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top,
-                      group_count, group_keep, group_top, scale, score_kind, chosen, weight);
+                      group_count, group_keep, group_top, scale, score_kind, normalize, chosen, weight);
     else return VM_ERR_UNSUPPORTED;
     return vm_launch_status();
 }

@@ -23,7 +23,8 @@ struct SkinnyParams {
     float* h;                    // residual [M, N]
     int I;                       // swiglu: rows of Wg (and of Wu)
     int store_act;               // bf16 store: 0, or 1 + the activation (VM_ACT_*) applied to the rounded product
-    int gate_act;                // swiglu: the activation of the gate (VM_ACT_SILU = 0, VM_ACT_GELU_TANH, VM_ACT_RELU_SQUARED)
+    int gate_act;                // swiglu: the activation of the gate (VM_ACT_SILU = 0, VM_ACT_GELU_TANH, VM_ACT_RELU_SQUARED), or GATE_CLAMPED
+    float limit, alpha;          // GATE_CLAMPED: its constants
     // rope_kv
     const int* positions; const int* seq_of_token; const int* block_table; int max_blocks;
     const float* inv_freq; int rot_dim;
@@ -42,6 +43,14 @@ __device__ __forceinline__ float skinny_gate(float z, int kind) {
     if (kind == VM_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     if (kind == VM_ACT_RELU_SQUARED) { const float r = fmaxf(z, 0.f); return r * r; }
     return z * (1.0f / (1.0f + expf(-z)));
+}
+
+constexpr int GATE_CLAMPED = -1;
+// the gated epilogue's value: act(g) u, or the clamped unit min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, +-limit) + 1)
+__device__ __forceinline__ float skinny_unit(const SkinnyParams& p, float g, float u) {
+    if (p.gate_act != GATE_CLAMPED) return skinny_gate(g, p.gate_act) * u;
+    g = fminf(g, p.limit);
+    return g * (1.0f / (1.0f + expf(-p.alpha * g))) * (fminf(fmaxf(u, -p.limit), p.limit) + 1.0f);
 }
 
 struct SkinnyCols { int nA, nB, head; };
@@ -281,7 +290,7 @@ __device__ __forceinline__ void skinny_run(const SkinnyParams& p, const int firs
                 if (two) o[nB + c] = res_b[it] + vB;
             } break;
             case EPI_SWIGLU: {
-                static_cast<__nv_bfloat16*>(p.out)[(size_t)row * p.out_stride + nA + c] = __float2bfloat16_rn(skinny_gate(vA, p.gate_act) * vB);
+                static_cast<__nv_bfloat16*>(p.out)[(size_t)row * p.out_stride + nA + c] = __float2bfloat16_rn(skinny_unit(p, vA, vB));
             } break;
             case EPI_ROPE_KV: {
                 const int pos = row_pos[it];

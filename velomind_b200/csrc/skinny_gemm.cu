@@ -201,6 +201,18 @@ VM_API int vm_skinny_gated(const void* A, int pro, const float* norm_w, float ep
     return skinny_dispatch(p, I / 8, stream);
 }
 
+// the same with the clamped unit: g = min(x Wg^T, limit), u = clamp(x Wu^T, -limit, limit), out = g sigmoid(alpha g) (u + 1)
+VM_API int vm_skinny_clamped(const void* A, int pro, const float* norm_w, float eps, const void* W, int M, int I, int K, float limit, float alpha, void* out,
+                             int* err, cudaStream_t stream) {
+    if (I % 8 != 0) return VM_ERR_UNSUPPORTED;
+    if (!(limit > 0.f)) return VM_ERR_BAD_ARG;
+    SkinnyParams p{};
+    p.err = err;
+    p.A = A; p.pro = pro; p.norm_w = norm_w; p.eps = eps; p.W = (const __nv_bfloat16*)W; p.M = M; p.N = 2 * I; p.K = K;
+    p.out = out; p.out_stride = I; p.I = I; p.epi = EPI_SWIGLU; p.tiles = 2; p.gate_act = GATE_CLAMPED; p.limit = limit; p.alpha = alpha;
+    return skinny_dispatch(p, I / 8, stream);
+}
+
 // the same with act = SiLU
 VM_API int vm_skinny_swiglu(const void* A, int pro, const float* norm_w, float eps, const void* W, int M, int I, int K,
                             void* out, int* err, cudaStream_t stream) {

@@ -301,7 +301,7 @@ skinny_stream_kernel(const SkinnyParams p) {
                         if (two) o[nB + c] = res_b + vB;
                     } break;
                     case EPI_SWIGLU: {
-                        static_cast<__nv_bfloat16*>(p.out)[(size_t)row * p.out_stride + nA + c] = __float2bfloat16_rn(skinny_gate(vA, p.gate_act) * vB);
+                        static_cast<__nv_bfloat16*>(p.out)[(size_t)row * p.out_stride + nA + c] = __float2bfloat16_rn(skinny_unit(p, vA, vB));
                     } break;
                     case EPI_ROPE_KV: {
                         float ya = vA, yb = vB;

@@ -408,6 +408,80 @@ int launch_norm_sum_norm(float* h, const T* y, const float* bias, const float* w
     return vm_launch_status();
 }
 
+// ------------------------------------------------------------------------------------------------ two sublayers on one input, joined
+// h += sa (ca a + ca2 a2) + sb b, value by value: a (and a2) what the mixer left, b the feed-forward's result, sa and sb [hid] float32.
+// a2 and b may be null, sa and sb too (1).  copy (activation dtype, may be null) receives the new h.
+template <typename T>
+__global__ void scaled_sum_vec_kernel(float* __restrict__ h, const T* __restrict__ a, float ca, const T* __restrict__ a2, float ca2, const float* __restrict__ sa,
+                                      const T* __restrict__ b, const float* __restrict__ sb, T* __restrict__ copy, long long n4, int hid4) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += (long long)gridDim.x * blockDim.x) {
+        const int col = 4 * (int)(i % hid4);
+        float4 v = ns_load4(h + 4 * i), x = ns_load4(a + 4 * i);
+        x.x *= ca; x.y *= ca; x.z *= ca; x.w *= ca;
+        if (a2) {
+            const float4 y = ns_load4(a2 + 4 * i);
+            x.x = fmaf(ca2, y.x, x.x); x.y = fmaf(ca2, y.y, x.y); x.z = fmaf(ca2, y.z, x.z); x.w = fmaf(ca2, y.w, x.w);
+        }
+        const float4 s = sa ? ns_load4(sa + col) : one;
+        x.x *= s.x; x.y *= s.y; x.z *= s.z; x.w *= s.w;
+        if (b) {
+            const float4 y = ns_load4(b + 4 * i), w = sb ? ns_load4(sb + col) : one;
+            x.x = fmaf(w.x, y.x, x.x); x.y = fmaf(w.y, y.y, x.y); x.z = fmaf(w.z, y.z, x.z); x.w = fmaf(w.w, y.w, x.w);
+        }
+        v.x += x.x; v.y += x.y; v.z += x.z; v.w += x.w;
+        ns_store4(h + 4 * i, v);
+        if (copy) ns_store4(copy + 4 * i, v);
+    }
+}
+
+template <typename T>
+__global__ void scaled_sum_kernel(float* __restrict__ h, const T* __restrict__ a, float ca, const T* __restrict__ a2, float ca2, const float* __restrict__ sa,
+                                  const T* __restrict__ b, const float* __restrict__ sb, T* __restrict__ copy, long long n, int hid) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const int col = (int)(i % hid);
+        float x = ca * vm_to_float(a[i]);
+        if (a2) x = fmaf(ca2, vm_to_float(a2[i]), x);
+        if (sa) x *= sa[col];
+        if (b) x = fmaf(sb ? sb[col] : 1.f, vm_to_float(b[i]), x);
+        const float v = h[i] + x;
+        h[i] = v;
+        if (copy) copy[i] = vm_from_float<T>(v);
+    }
+}
+
+template <typename T>
+int launch_scaled_sum(float* h, const T* a, float ca, const T* a2, float ca2, const float* sa, const T* b, const float* sb, T* copy, int T_, int hid,
+                      cudaStream_t stream) {
+    const uintptr_t at = (uintptr_t)h | (uintptr_t)a | (uintptr_t)a2 | (uintptr_t)sa | (uintptr_t)b | (uintptr_t)sb | (uintptr_t)copy;
+    const bool vec = hid % 4 == 0 && at % 16 == 0;
+    const long long n = (long long)T_ * hid / (vec ? 4 : 1), want = (n + 255) / 256;
+    const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+    if (vec) vm_launch_pdl(scaled_sum_vec_kernel<T>, grid, dim3(256), 0, stream, h, a, ca, a2, ca2, sa, b, sb, copy, n, hid / 4);
+    else vm_launch_pdl(scaled_sum_kernel<T>, grid, dim3(256), 0, stream, h, a, ca, a2, ca2, sa, b, sb, copy, n, hid);
+    return vm_launch_status();
+}
+
+// ------------------------------------------------------------------------------------------------ a token's own row, gated
+// out[t, i] = gelu_tanh(z[t, i]) * table[token_t, off + i]; z float32 [T, ldz], table rows of ld_table values in W.  A token outside the
+// table reads its first row (the embedding, which reads the same token, reports it).
+template <typename W, typename T>
+__global__ void gated_token_rows_kernel(const float* __restrict__ z, int ldz, const int* __restrict__ tokens, const W* __restrict__ table, long long ld_table,
+                                        int off, int vocab, T* __restrict__ out, int n, long long total) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / n;
+        const int c = (int)(i - t * n), id = tokens[t];
+        const float v = z[t * ldz + c], e = vm_to_float(table[(size_t)(id >= 0 && id < vocab ? id : 0) * ld_table + off + c]);
+        out[i] = vm_from_float<T>(0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))) * e);
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ polynomial activation with unit-rms powers
 // one block per token; z [T, n] in Z (float32 or the activation dtype), out in T
 template <typename Z, typename T>
@@ -630,6 +704,34 @@ VM_API int vm_norm_sum_norm(float* h, const void* y, const float* bias, const fl
     if (act_dtype == VM_BF16)
         return launch_norm_sum_norm<__nv_bfloat16>(h, (const __nv_bfloat16*)y, bias, w_out, eps_out, w_in, eps_in, (__nv_bfloat16*)out, rows, n, hid, stream);
     return VM_ERR_UNSUPPORTED;
+}
+
+VM_API int vm_scaled_sum(float* h, const void* a, float ca, const void* a2, float ca2, const float* sa, const void* b, const float* sb, void* copy, int T, int hid,
+                         int act_dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (hid <= 0 || !a) return VM_ERR_BAD_ARG;
+    if (act_dtype == VM_F32)
+        return launch_scaled_sum<float>(h, (const float*)a, ca, (const float*)a2, ca2, sa, (const float*)b, sb, (float*)copy, T, hid, stream);
+    if (act_dtype == VM_BF16)
+        return launch_scaled_sum<__nv_bfloat16>(h, (const __nv_bfloat16*)a, ca, (const __nv_bfloat16*)a2, ca2, sa, (const __nv_bfloat16*)b, sb,
+                                                (__nv_bfloat16*)copy, T, hid, stream);
+    return VM_ERR_UNSUPPORTED;
+}
+
+VM_API int vm_gated_token_rows(const float* z, int ldz, const int* tokens, const void* table, int table_dtype, long long ld_table, int off, int vocab, void* out,
+                               int n, int T, int act_dtype, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (n <= 0 || ldz < n || off < 0 || ld_table < off + n || vocab <= 0) return VM_ERR_BAD_ARG;
+    const long long total = (long long)T * n, want = (total + 255) / 256;
+    const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+#define VM_GTR(W, T_) \
+    vm_launch_pdl(gated_token_rows_kernel<W, T_>, grid, dim3(256), 0, stream, z, ldz, tokens, (const W*)table, ld_table, off, vocab, (T_*)out, n, total)
+    if (table_dtype == VM_F32 && act_dtype == VM_F32) VM_GTR(float, float);
+    else if (table_dtype == VM_F32 && act_dtype == VM_BF16) VM_GTR(float, __nv_bfloat16);
+    else if (table_dtype == VM_BF16 && act_dtype == VM_BF16) VM_GTR(__nv_bfloat16, __nv_bfloat16);
+    else return VM_ERR_UNSUPPORTED;
+#undef VM_GTR
+    return vm_launch_status();
 }
 
 // One token per sequence (token s is sequence s's): h += rmsnorm(y) * w, then out = h + conv(h) as vm_input_conv does for such a step,

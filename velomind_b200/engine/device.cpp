@@ -149,10 +149,14 @@ DeviceTensor BindContext::upload_stacked(const std::vector<const HostTensor*>& p
 }
 
 DeviceTensor BindContext::upload_scaled(const HostTensor& t, float factor) {
+    return upload_mapped(t, [factor](float v) { return v * factor; });
+}
+
+DeviceTensor BindContext::upload_mapped(const HostTensor& t, const std::function<float(float)>& map) {
     const std::vector<uint8_t> bytes = converted(t, DType::F32);
     std::vector<float> values(bytes.size() / sizeof(float));
     std::memcpy(values.data(), bytes.data(), values.size() * sizeof(float));
-    for (float& v : values) v *= factor;
+    for (float& v : values) v = map(v);
     DeviceTensor d = upload_floats(values);
     d.shape = t.shape;
     return d;
@@ -510,6 +514,17 @@ void attention(StepContext& ctx, const void* q, int q_row_stride, const KVView& 
           "attention_generic", s);
 }
 
+int selective_piece_tokens(const StepContext& ctx, int C) {
+    if (ctx.T_cap < 64) return 0;
+    // a warp takes 8 channels; with about one warp for each of an SM's four schedulers one pass over the tokens is as fast as the pieces'
+    // two passes and their carry
+    const long long warps = static_cast<long long>(ctx.B_cap) * ((C + 7) / 8), want = 4ll * sm_count();
+    if (10 * warps >= 6 * want) return 0;
+    const long long pieces = (3 * want + warps - 1) / warps;      // per sequence of equal length: about three warps for each scheduler
+    const long long tokens = (ctx.T_cap / std::max(1, ctx.B_cap) + pieces - 1) / pieces;
+    return static_cast<int>(std::max<long long>(32, (tokens + 31) / 32 * 32));
+}
+
 void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const KVView& kv, void* out, int H, int Hkv, int Dk, int Dv, float scale,
                       const BiasedMask& mask) {
     cudaStream_t s = ctx.stream;
@@ -519,7 +534,7 @@ void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const K
     if (ctx.act_dtype == DType::BF16 && ctx.one_token_each && Dk <= 1024 && Dv <= 256 && H <= 65535) {
         Timed t("attention_biased_decode_bf16", s);
         check(vm_attention_sink_decode_bf16(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, mask.rel, mask.bucket_of,
-                                            mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.B, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
+                                            mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.B, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first, mask.chunk,
                                             kv.n_pages, ctx.err, s),
               "attention_biased_decode_bf16", s);
         return;
@@ -530,13 +545,13 @@ void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const K
         Timed t("attention_biased_prefill_bf16", s);
         check(vm_attention_sink_prefill_bf16(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, ctx.cu_tokens, ctx.B,
                                              static_cast<int>(tiles), mask.rel, mask.bucket_of, mask.far, mask.rows, mask.sink, mask.slopes, mask.v_row_stride, out, H,
-                                             Hkv, Dk, Dv, scale, mask.window, mask.keep_first, kv.n_pages, ctx.err, s),
+                                             Hkv, Dk, Dv, scale, mask.window, mask.keep_first, mask.chunk, kv.n_pages, ctx.err, s),
               "attention_biased_prefill_bf16", s);
         return;
     }
     Timed t("attention_biased_generic", s);
     check(vm_attention_sink_generic(q, q_row_stride, kv.k_pages, kv.v_pages, kv.block_table, kv.table_width, ctx.positions, ctx.seq_of_token, mask.rel,
-                                    mask.bucket_of, mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.T, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first,
+                                    mask.bucket_of, mask.far, mask.sink, mask.slopes, mask.v_row_stride, out, ctx.T, H, Hkv, Dk, Dv, scale, mask.window, mask.keep_first, mask.chunk,
                                     kv.n_pages, code(ctx.act_dtype), ctx.err, s),
           "attention_biased_generic", s);
 }

@@ -134,9 +134,10 @@ std::vector<CacheNeed> DecoderModel::cache_needs() const {
         if (reader.kv_heads != kept.kv_heads || reader.key_dim != kept.key_dim || reader.value_dim != kept.value_dim)
             throw ConfigError(format("a layer reads the keys and values of run %d, which have other sizes than its own", e.cache_of));
         if (kept.kind == CacheNeed::All) continue;
-        if (reader.kind == CacheNeed::All) {
+        if (kept.kind == CacheNeed::Chunk && reader.kind == CacheNeed::Chunk && kept.chunk == reader.chunk) continue;
+        if (reader.kind == CacheNeed::All || reader.kind == CacheNeed::Chunk || kept.kind == CacheNeed::Chunk) {      // (chunks and windows, or unlike chunks: everything)
             kept.kind = CacheNeed::All;
-            kept.window = kept.keep_first = 0;
+            kept.window = kept.keep_first = kept.chunk = 0;
         } else {
             kept.window = std::max(kept.window, reader.window);
             kept.keep_first = std::max(kept.keep_first, reader.keep_first);
@@ -192,6 +193,7 @@ void DecoderModel::forward(StepContext& ctx) {
     float* h = static_cast<float*>(ctx.take_tokens(hid * S, DType::F32));      // copy s of the stream: [T, hid] at h + s * stream_stride
     ctx.run = static_cast<int>(plan.schedule.size());                          // the embedding's own state area, if it keeps one
     embedding->forward(ctx, ctx.tokens, h);
+    ctx.token_rows = embedding->token_rows();
     for (int s = 1; s < S; ++s)                                               // every copy starts as the embedding's output
         ops::cuda_check(cudaMemcpyAsync(h + s * ctx.stream_stride, h, static_cast<size_t>(ctx.T) * hid * sizeof(float), cudaMemcpyDeviceToDevice, ctx.stream),
                         "copying the residual stream");

@@ -146,6 +146,26 @@ inline void gated_activation(const void* gate_up, void* out, int T, int I, int k
     check(vm_gated_activation(gate_up, out, T, I, kind, code(act), s), "gated_activation", s);
 }
 
+inline void clamped_unit(const void* gate_up, void* out, int T, int I, float limit, float alpha, DType act, cudaStream_t s) {
+    Timed t("clamped_unit", s);
+    check(vm_clamped_unit(gate_up, out, T, I, limit, alpha, code(act), s), "clamped_unit", s);
+}
+
+// two sublayers on one input, joined: h += sa (ca a + ca2 a2) + sb b (a2, sa, b, sb may be null); copy (or null) receives the new h
+inline void scaled_sum(float* h, const void* a, float ca, const void* a2, float ca2, const float* sa, const void* b, const float* sb, void* copy,
+                       const StepContext& ctx) {
+    Timed t("scaled_sum", ctx.stream);
+    check(vm_scaled_sum(h, a, ca, a2, ca2, sa, b, sb, copy, ctx.T, ctx.hidden, code(ctx.act_dtype), ctx.stream), "scaled_sum", ctx.stream);
+}
+
+// out[t, i] = gelu_tanh(z[t, i]) * table[token_t, off + i] for the step's tokens
+inline void gated_token_rows(const float* z, int ldz, const DeviceTensor& table, int off, int n, void* out, const StepContext& ctx) {
+    Timed t("gated_token_rows", ctx.stream);
+    check(vm_gated_token_rows(z, ldz, ctx.tokens, table.ptr, code(table.dtype), table.cols(), off, static_cast<int>(table.rows()), out, n, ctx.T,
+                              code(ctx.act_dtype), ctx.stream),
+          "gated_token_rows", ctx.stream);
+}
+
 inline void convert(const void* in, DType in_dtype, void* out, DType out_dtype, long long n, cudaStream_t s) {
     Timed t("convert", s);
     check(vm_convert(in, code(in_dtype), out, code(out_dtype), n, s), "convert", s);
@@ -250,11 +270,11 @@ struct ExpertKind {
 };
 
 inline void expert_router_scored(const void* x, const float* norm_w, float eps, const float* w_router, const float* correction, int T, int hidden,
-                                 int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, int* chosen, float* weight,
-                                 DType act, cudaStream_t s) {
+                                 int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, bool normalize, int* chosen,
+                                 float* weight, DType act, cudaStream_t s) {
     Timed t("expert_router", s);
-    check(vm_expert_router_groups(x, norm_w, eps, w_router, correction, T, hidden, n_out, top, group_count, group_keep, group_top, scale, score_kind, chosen,
-                                  weight, code(act), s),
+    check(vm_expert_router_groups(x, norm_w, eps, w_router, correction, T, hidden, n_out, top, group_count, group_keep, group_top, scale, score_kind,
+                                  normalize ? 1 : 0, chosen, weight, code(act), s),
           "expert_router", s);
 }
 
@@ -295,6 +315,7 @@ struct BiasedMask {
     const float* rel = nullptr;         // device float32 [rows, H], or null: no bias
     const int* bucket_of = nullptr;     // device int32 [far + 1]
     int far = 0, rows = 0, window = 0, keep_first = 0;
+    int chunk = 0;                      // > 0: only keys of the query's own chunk of so many places (and kept ones)
     const float* sink = nullptr;        // device float32 [H], or null: exp(sink[h]) joins head h's softmax denominator
     const float* slopes = nullptr;      // device float32 [H], or null: slopes[h] (i - j) comes off head h's score of key j at place i
     int v_row_stride = 0;               // elements between neighbouring tokens' value rows (0: Dv); Dk with the key pool as value pool: values inside keys
@@ -308,7 +329,8 @@ constexpr int SSM_CHUNKS_FROM_TOKENS = 64;      // a step's capacity from which 
 inline void ssm_mixer(const void* proj, int ld, const float* taps, const float* conv_bias, const float* dt_bias, const float* A_log, const float* Dskip,
                       const float* norm_w, float eps, StepContext& ctx, void* out, int H, int P, int N, int G, int K, int parts) {
     Timed t("ssm_mixer", ctx.stream);
-    if (!ctx.state() || ctx.state_floats() < vm_ssm_state_floats(H, P, N, G, K)) throw CacheError("ssm: the cache holds no state area of this layer's size");
+    if (!ctx.state() || ctx.state_floats() < ctx.state_offset + vm_ssm_state_floats(H, P, N, G, K))
+        throw CacheError("ssm: the cache holds no state area of this layer's size");
     const long long C = static_cast<long long>(H) * P + 2ll * G * N;
     void* xbc = ctx.take_tokens(C, ctx.act_dtype);
     float* y = static_cast<float*>(ctx.take_tokens(static_cast<long long>(H) * P, DType::F32));
@@ -321,8 +343,8 @@ inline void ssm_mixer(const void* proj, int ld, const float* taps, const float* 
         scratch = static_cast<float*>(ctx.take(vm_ssm_chunk_scratch_floats(ctx.T_cap, ctx.T_cap / 64 + ctx.B_cap, H, P, N), DType::F32));
         for (int b = 0; b < ctx.B; ++b) n_chunks += (ctx.host_cu_tokens[b + 1] - ctx.host_cu_tokens[b] + 63) / 64;
     }
-    check(vm_ssm_mixer(proj, ld, taps, conv_bias, dt_bias, A_log, Dskip, norm_w, eps, ctx.state(), ctx.state_floats(), ctx.positions, ctx.seq_of_token,
-                       ctx.cu_tokens, ctx.slots, xbc, y, out, scratch, n_chunks, ctx.one_token_each ? 1 : 0, ctx.T, ctx.B, H, P, N, G, K, parts,
+    check(vm_ssm_mixer(proj, ld, taps, conv_bias, dt_bias, A_log, Dskip, norm_w, eps, ctx.state() + ctx.state_offset, ctx.state_floats(), ctx.positions,
+                       ctx.seq_of_token, ctx.cu_tokens, ctx.slots, xbc, y, out, scratch, n_chunks, ctx.one_token_each ? 1 : 0, ctx.T, ctx.B, H, P, N, G, K, parts,
                        code(ctx.act_dtype), ctx.stream),
           "ssm_mixer", ctx.stream);
     counters().own_launches += ctx.one_token_each ? 2 : (chunks ? 5 : (K > 1 ? 3 : 2));
@@ -411,6 +433,12 @@ inline void skinny_gated(const void* x, const float* norm_w, float eps, const De
     check(vm_skinny_gated(x, norm_w ? 1 : 0, norm_w, eps, W.ptr, M, I, static_cast<int>(W.cols()), act, out, err, s), "skinny_gated", s);
 }
 
+inline void skinny_clamped(const void* x, const float* norm_w, float eps, const DeviceTensor& W, int M, int I, float limit, float alpha, void* out, int* err,
+                           cudaStream_t s) {
+    Timed t("skinny_gated", s);
+    check(vm_skinny_clamped(x, norm_w ? 1 : 0, norm_w, eps, W.ptr, M, I, static_cast<int>(W.cols()), limit, alpha, out, err, s), "skinny_gated", s);
+}
+
 inline void skinny_qkv_rope(const void* x, const float* norm_w, float eps, const DeviceTensor& W, void* q_out, const StepContext& ctx, const KVView& kv,
                             const RotaryTable& rot, int H, int Hkv, int D) {
     Timed t("skinny_qkv_rope", ctx.stream);
@@ -473,13 +501,13 @@ inline void need_state(const StepContext& ctx, long long floats, const char* who
     if (!ctx.state() || ctx.state_floats() < ctx.state_offset + floats) throw CacheError(std::string(who) + ": the cache holds no state area of this part's size");
 }
 
-inline void embed_pairs(const DeviceTensor& table, const DeviceTensor& pairs, long long buckets, long long mul_prev, long long mul_cur, StepContext& ctx,
-                        float* out) {
+inline void embed_pairs(const DeviceTensor& table, const DeviceTensor& pairs, long long buckets, long long mul_prev, long long mul_cur, float scale,
+                        StepContext& ctx, float* out) {
     Timed t("embed_pairs", ctx.stream);
     need_state(ctx, 1, "embedding");
     check(vm_embed_pairs(table.ptr, pairs.ptr, code(table.dtype), ctx.tokens, ctx.positions, ctx.seq_of_token, ctx.cu_tokens, ctx.slots,
                          reinterpret_cast<int*>(ctx.state() + ctx.state_offset), ctx.state_floats(), out, ctx.T, ctx.B, ctx.hidden,
-                         static_cast<int>(table.rows()), buckets, mul_prev, mul_cur, ctx.one_token_each ? 1 : 0, ctx.err, ctx.stream),
+                         static_cast<int>(table.rows()), buckets, mul_prev, mul_cur, scale, ctx.one_token_each ? 1 : 0, ctx.err, ctx.stream),
           "embed_pairs", ctx.stream);
     if (!ctx.one_token_each) ++counters().own_launches;
 }
@@ -557,6 +585,48 @@ inline void decayed_memory(float* proj, int ld, const MemoryArgs& a, StepContext
 inline void memory_output(const float* o, const float* g, int ldg, const float* w, float eps, void* out, int T, int H, int Dv, DType act, cudaStream_t s) {
     Timed t("memory_output", s);
     check(vm_memory_output(o, g, ldg, w, eps, out, T, H, Dv, code(act), s), "memory_output", s);
+}
+
+// the selective state-space mixer over the running part's state: S [C, N], then the convolution's kept inputs
+inline void short_conv_silu(const void* proj, int ld, int u_col, const float* taps, const float* bias, int conv_off, StepContext& ctx, int C, int K, void* out) {
+    Timed t("short_conv_silu", ctx.stream);
+    need_state(ctx, conv_off + static_cast<long long>(K - 1) * C, "convolution");
+    check(vm_short_conv_silu(proj, ld, u_col, taps, bias, ctx.state() + ctx.state_offset, ctx.state_floats(), conv_off, ctx.positions, ctx.seq_of_token,
+                             ctx.cu_tokens, ctx.slots, ctx.one_token_each ? 1 : 0, ctx.T, ctx.B, C, K, out, code(ctx.act_dtype), ctx.stream),
+          "short_conv_silu", ctx.stream);
+    if (!ctx.one_token_each && K > 1) ++counters().own_launches;
+}
+inline void selective_step(const void* x, const float* r, int ldr, const DeviceTensor& w_dt, int rank, const void* z, int ldz, const float* dt_bias,
+                           const float* A2, const float* D, StepContext& ctx, void* out, int C, int N) {
+    Timed t("selective_step", ctx.stream);
+    need_state(ctx, static_cast<long long>(C) * N, "selective_scan");
+    check(vm_selective_step(x, r, ldr, w_dt.ptr, code(w_dt.dtype), rank, z, ldz, dt_bias, A2, D, ctx.state() + ctx.state_offset, ctx.state_floats(), ctx.slots,
+                            out, ctx.B, C, N, code(ctx.act_dtype), ctx.stream),
+          "selective_step", ctx.stream);
+}
+// tokens per piece of a prompt's scan (0: one pass), from the step's capacity alone, so that every step of a bucket asks for the same scratch
+int selective_piece_tokens(const StepContext& ctx, int C);
+inline void selective_scan(const void* x, const float* dt, int ldt, const float* r, int ldr, int b_col, const void* z, int ldz, const float* dt_bias,
+                           const float* A2, const float* D, StepContext& ctx, void* out, int C, int N) {
+    Timed t("selective_scan", ctx.stream);
+    need_state(ctx, static_cast<long long>(C) * N, "selective_scan");
+    const int piece = selective_piece_tokens(ctx, C);
+    float* scratch = nullptr;
+    int n_pieces = ctx.B;
+    if (piece > 0) {
+        scratch = static_cast<float*>(ctx.take(vm_selective_scratch_floats(ctx.T_cap / piece + ctx.B_cap, C, N), DType::F32));
+        n_pieces = 0;
+        for (int b = 0; b < ctx.B; ++b) n_pieces += (ctx.host_cu_tokens[b + 1] - ctx.host_cu_tokens[b] + piece - 1) / piece;
+    }
+    check(vm_selective_scan(x, dt, ldt, r, ldr, b_col, z, ldz, dt_bias, A2, D, ctx.state() + ctx.state_offset, ctx.state_floats(), ctx.cu_tokens, ctx.slots, out,
+                            scratch, piece, n_pieces, ctx.B, C, N, code(ctx.act_dtype), ctx.stream),
+          "selective_scan", ctx.stream);
+    if (scratch) counters().own_launches += 2;      // three kernels
+    ctx.give(scratch);
+}
+inline void take_columns(const float* src, int ld, int col, void* dst, int n, StepContext& ctx) {
+    Timed t("take_columns", ctx.stream);
+    check(vm_take_columns(src, ld, col, dst, n, ctx.T, code(ctx.act_dtype), ctx.stream), "take_columns", ctx.stream);
 }
 
 // the gated delta rule over the running part's state: from the projections (layout as vm_delta_step) to the gated, normed heads in `out`

@@ -49,6 +49,8 @@ int vm_swiglu(const void* gate_up, void* out, int T, int I, int act_dtype, cudaS
 int vm_convert(const void* in, int in_dtype, void* out, int out_dtype, long long n, cudaStream_t stream);
 // out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i] for the activation `kind` (VM_ACT_*)
 int vm_gated_activation(const void* gate_up, void* out, int T, int I, int kind, int act_dtype, cudaStream_t stream);
+// the clamped gated unit: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(alpha g) (u + 1)
+int vm_clamped_unit(const void* gate_up, void* out, int T, int I, float limit, float alpha, int act_dtype, cudaStream_t stream);
 
 // ---- latent_cache.cu: the norms of a latent-attention layer's two down projections and the cache write of the key/value latent
 // down float32 [T, ld]: columns [0, q_rank) and, if `pages` is given, [q_rank, q_rank + kv_rank); cq [T, q_rank] and the
@@ -74,6 +76,12 @@ int vm_norm_residual_add(float* h, const void* y, long long ld, int y_dtype, con
 int vm_norm_residual_conv_step(float* h, const void* y, long long ld, int y_dtype, const float* w, int B, int hid, float eps, const float* taps,
                                float* state, long long state_stride, int state_offset, const int* slots, void* out, int K, int act_dtype,
                                cudaStream_t stream);
+// h += sa (ca a + ca2 a2) + sb b value by value (a2, sa, b, sb may be null: not there, or 1); copy (null: none) receives the new h in act_dtype
+int vm_scaled_sum(float* h, const void* a, float ca, const void* a2, float ca2, const float* sa, const void* b, const float* sb, void* copy, int T, int hid,
+                  int act_dtype, cudaStream_t stream);
+// out[t, i] = gelu_tanh(z[t, i]) * table[token_t, off + i]
+int vm_gated_token_rows(const float* z, int ldz, const int* tokens, const void* table, int table_dtype, long long ld_table, int off, int vocab, void* out, int n,
+                        int T, int act_dtype, cudaStream_t stream);
 // a N(z) + b N(z^2) + c N(z^3) + e per token, N: division by the root mean square over the token's n values; coef float32 [4]
 int vm_polynorm(const void* z, int z_dtype, const float* coef, void* out, int T, int n, float eps, int act_dtype, cudaStream_t stream);
 int vm_rotate_slice(const void* src, long long src_ld, int src_head, int src_off, void* dst, long long dst_ld, int dst_head, int dst_off,
@@ -135,7 +143,7 @@ int vm_expert_router_scores(const void* x, const float* norm_w, float eps, const
                             cudaStream_t stream);      // vm_expert_router_scored with the kind of score (VM_SCORE_*) as an argument
 // the same with the number of a group's largest scores that make up the group's score (1: its largest; 2: the sum of its two largest)
 int vm_expert_router_groups(const void* x, const float* norm_w, float eps, const float* w_router, const float* correction, int T, int hidden,
-                            int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, int* chosen,
+                            int n_out, int top, int group_count, int group_keep, int group_top, float scale, int score_kind, int normalize, int* chosen,
                             float* weight, int act_dtype, cudaStream_t stream);
 
 // ---- attention_biased.cu: windowed attention with kept first tokens and a learned bias by bucketed distance; keys of Dk, values of Dv
@@ -155,18 +163,19 @@ int vm_attention_biased_generic(const void* q, int q_row_stride, const void* kpa
 // The same attention with a sink and with values that may lie inside the key rows.  sink float32 [H] (null: none): exp(sink[h]) is one
 // more term of head h's softmax denominator, without a key or a value, not scaled.  v_row_stride: elements between the value rows of
 // neighbouring tokens in `vpages` (0: Dv); with vpages == kpages and v_row_stride == Dk a token's value is the first Dv values of its key row.
+// chunk > 0: of the keys the window leaves, a query at position p sees those from chunk floor(p / chunk) on (and the kept ones).
 int vm_attention_sink_generic(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                               const int* positions, const int* seq_of_token, const float* rel, const int* bucket_of, int far, const float* sink, const float* slopes,
                               int v_row_stride, void* out, int n_tokens, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first,
-                              int n_pages, int act_dtype, int* err, cudaStream_t stream);
+                              int chunk, int n_pages, int act_dtype, int* err, cudaStream_t stream);
 int vm_attention_sink_prefill_fits(int Dk, int Dv, int values_in_keys);
 int vm_attention_sink_prefill_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                                    const int* positions, const int* cu_tokens, int B, int n_tiles, const float* rel, const int* bucket_of, int far,
                                    int rel_rows, const float* sink, const float* slopes, int v_row_stride, void* out, int H, int Hkv, int Dk, int Dv, float scale, int window,
-                                   int keep_first, int n_pages, int* err, cudaStream_t stream);
+                                   int keep_first, int chunk, int n_pages, int* err, cudaStream_t stream);
 int vm_attention_sink_decode_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table, int max_blocks,
                                   const int* positions, const float* rel, const int* bucket_of, int far, const float* sink, const float* slopes, int v_row_stride, void* out,
-                                  int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err,
+                                  int B, int H, int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int chunk, int n_pages, int* err,
                                   cudaStream_t stream);
 
 // ---- attention_biased_fast.cu: the same attention in bfloat16: prompts on mma.sync tiles (keys and values of the sizes that
@@ -179,6 +188,26 @@ int vm_attention_biased_prefill_bf16(const void* q, int q_row_stride, const void
 int vm_attention_biased_decode_bf16(const void* q, int q_row_stride, const void* kpages, const void* vpages, const int* block_table,
                                     int max_blocks, const int* positions, const float* rel, const int* bucket_of, int far, void* out, int B, int H,
                                     int Hkv, int Dk, int Dv, float scale, int window, int keep_first, int n_pages, int* err, cudaStream_t stream);
+
+// ---- selective_scan.cu: a selective state-space mixer with a state of N values per channel and an input-dependent step size
+long long vm_selective_state_floats(int C, int N, int K);
+long long vm_selective_scratch_floats(int n_pieces, int C, int N);
+int vm_selective_max_state();      // the largest N the prompt kernel takes
+// the short convolution with SiLU in front of it (or of another recurrence): columns [u_col, u_col + C) of proj, the last K - 1 inputs kept
+// in slot s's floats from state + s * state_floats + conv_off on
+int vm_short_conv_silu(const void* proj, int ld, int u_col, const float* taps, const float* bias, float* state, int state_floats, int conv_off,
+                       const int* positions, const int* seq_of_token, const int* cu_tokens, const int* slots, int one_token_each, int T, int B, int C, int K,
+                       void* out, int act_dtype, cudaStream_t stream);
+// prompts: dt float32 [T, ldt] before bias and softplus, B | C at columns b_col of r float32 [T, ldr], A2 = A log2(e) [C, N]; scratch null: one
+// pass over the tokens, else pieces of `piece` tokens side by side
+int vm_selective_scan(const void* x, const float* dt, int ldt, const float* r, int ldr, int b_col, const void* z, int ldz, const float* dt_bias,
+                      const float* A2, const float* D, float* state, long long state_stride, const int* cu_tokens, const int* slots, void* out, float* scratch,
+                      int piece, int n_pieces, int B, int C, int N, int act_dtype, cudaStream_t stream);
+// one token per sequence: r rows [rank | B | C], the step size's product included (w_dt [C, rank] in w_dtype)
+int vm_selective_step(const void* x, const float* r, int ldr, const void* w_dt, int w_dtype, int rank, const void* z, int ldz, const float* dt_bias,
+                      const float* A2, const float* D, float* state, long long state_stride, const int* slots, void* out, int B, int C, int N, int act_dtype,
+                      cudaStream_t stream);
+int vm_take_columns(const float* src, int ld, int col, void* dst, int n, int T, int act_dtype, cudaStream_t stream);      // dst [T, n] = columns of src
 
 // ---- ssm.cu: a selective state-space mixer (short causal convolution, matrix-state recurrence, gated group norm)
 long long vm_ssm_state_floats(int H, int P, int N, int G, int K);
@@ -244,6 +273,9 @@ int vm_skinny_swiglu(const void* A, int pro, const float* norm_w, float eps, con
                      int* err, cudaStream_t stream);
 int vm_skinny_gated(const void* A, int pro, const float* norm_w, float eps, const void* W, int M, int I, int K, int act, void* out,
                     int* err, cudaStream_t stream);      // vm_skinny_swiglu with the gate's activation (VM_ACT_*) as an argument
+// ... with the clamped unit (vm_clamped_unit) instead of act(gate) * up
+int vm_skinny_clamped(const void* A, int pro, const float* norm_w, float eps, const void* W, int M, int I, int K, float limit, float alpha, void* out, int* err,
+                      cudaStream_t stream);
 void vm_skinny_variant(int variant);       // 0 choose by size, 1 / 2 force one of the two kernels (tests, measurements)
 int vm_skinny_qkv_rope(const void* A, int pro, const float* norm_w, float eps, const void* W, int M, int K, void* q_out,
                        const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
@@ -268,11 +300,11 @@ int vm_tc_qkv_rope(const void* A, long long lda, const void* W, int M, int K, vo
 int vm_streams_step(float* h, long long stride, int S, const void* y, const float* mix, const float* w_out, const float* w_in, const float* norm_w,
                     float eps, void* out, int T, int hid, int act_dtype, cudaStream_t stream);
 int vm_streams_sum_rows(float* h, long long stride, int S, const int* rows, int n_rows, int hid, cudaStream_t stream);   // copy 0 <- the sum, at `rows`
-// out[t] = table[token] + pairs[(previous * mul_prev + token * mul_cur) mod buckets], row `buckets` for a sequence's first token;
+// out[t] = scale * table[token] + pairs[(previous * mul_prev + token * mul_cur) mod buckets], row `buckets` for a sequence's first token;
 // `last`: an int32 word per slot (last_stride words apart) that keeps the token before the next step's first one
 int vm_embed_pairs(const void* table, const void* pairs, int table_dtype, const int* tokens, const int* positions, const int* seq_of_token,
                    const int* cu_tokens, const int* slots, int* last, long long last_stride, float* out, int T, int B, int hid, int vocab,
-                   long long buckets, long long mul_prev, long long mul_cur, int one_token_each, int* err, cudaStream_t stream);
+                   long long buckets, long long mul_prev, long long mul_cur, float scale, int one_token_each, int* err, cudaStream_t stream);
 
 // ---- mixer_prep.cu: from an attention mixer's projections to its attention kernel (bias, short convolution over time with kept rows,
 // norm over the whole projection, rotary positions, cache write), and gates, biases and joins behind it

@@ -280,6 +280,7 @@ public:
     DeviceTensor upload(const HostTensor& t, DType as);
     // rows of several matrices, one tensor; its rows are filled up with zeros to a multiple of `row_multiple`
     DeviceTensor upload_stacked(const std::vector<const HostTensor*>& parts, DType as, int row_multiple = 1);
+    DeviceTensor upload_mapped(const HostTensor& t, const std::function<float(float)>& map);   // float32, every value through `map`
     DeviceTensor upload_scaled(const HostTensor& t, float factor);                         // float32, every value times `factor`
     DeviceTensor upload_floats(const std::vector<float>& values);
     DeviceTensor upload_ints(const std::vector<int>& values);
@@ -314,15 +315,16 @@ private:
 
 // What one run of a mixer keeps per sequence.
 struct CacheNeed {
-    enum Kind { None, All, Window } kind = None;   // every earlier key/value; the last `window`; nothing
+    enum Kind { None, All, Window, Chunk } kind = None;   // nothing; every earlier key/value; the last `window`; those of the newest chunk of places
     int kv_heads = 0;
     int key_dim = 0, value_dim = 0;                // per head; they may differ; value_dim 0: one row per token only
     int window = 0;
     int keep_first = 0;                            // a window group keeps the pages of the first `keep_first` tokens for good
+    int chunk = 0;                                 // places per chunk of a chunk group, counted from the sequence's start
     int state_floats = 0;                          // fixed-size float32 state per sequence (0: none)
     bool same_group(const CacheNeed& o) const {
         return kind == o.kind && kv_heads == o.kv_heads && key_dim == o.key_dim && value_dim == o.value_dim && window == o.window &&
-               keep_first == o.keep_first;
+               keep_first == o.keep_first && chunk == o.chunk;
     }
 };
 
@@ -332,7 +334,7 @@ public:
     PageBook(const CacheNeed& need, int n_pages, int max_slots, int max_blocks);
     int pages_needed(int slot, int new_len) const;
     void ensure(int slot, int new_len);            // give `slot` pages so that tokens [0, new_len) have a place
-    void trim(int slot, int length);               // a window group gives back the pages no later query can reach
+    void trim(int slot, int length);               // a window or chunk group gives back the pages no later query can reach
     void release(int slot);
     const int* table_row(int slot) const { return &table_[static_cast<size_t>(slot) * max_blocks]; }
     CacheNeed need;
@@ -489,6 +491,14 @@ struct StepContext {
         if (takes_row_bias) row_bias = bias;
         return takes_row_bias;
     }
+    // A mixer whose result is a weighted sum of two (two mixers side by side) may leave the sum to a wiring that can carry it out: the wiring
+    // says so with `takes_two_terms` before it runs the mixer, and finds, if the mixer took the offer, the second result (a buffer of the
+    // workspace, to be given back) in `second_term` and the weights of both afterwards.
+    bool takes_two_terms = false;
+    void* second_term = nullptr;
+    float first_weight = 1.f, second_weight = 0.f;
+    // Rows per token that a model keeps beside its embedding (all layers' side by side, in one table), or null
+    const DeviceTensor* token_rows = nullptr;
     // ... or, in a model with several copies of the stream, through the mixing its layer left with it: copy t becomes
     // sum_s pending_mix[s, t] x_s + pending_out[t] * delta (device float32 [streams, streams] and [streams])
     const float *pending_mix = nullptr, *pending_out = nullptr;
@@ -587,6 +597,8 @@ public:
     // float32 words the embedding keeps per sequence (the token before the step's first one); while it runs, `ctx.state()` is that
     // area, which lies behind the schedule's own: a state area numbered schedule.size()
     virtual int state_floats() const { return 0; }
+    // a table [vocab, n] of further rows per token, which layers read a part of by the token's id (null: none)
+    virtual const DeviceTensor* token_rows() const { return nullptr; }
 };
 
 class Head : public Part {

@@ -1,6 +1,6 @@
 // Arrangements: how a layer wires its norms, mixer, feed-forward and the residual stream.
 #include "args.h"
-#include "../engine/ops.h"
+#include "linear.h"
 
 namespace vmb {
 
@@ -338,6 +338,125 @@ private:
     DeviceTensor out_[2];
 };
 
+// One norm and both sublayers on its output: x = norm(h); h += mixer(x) * s1 + feed_forward(x) * s2, with s1 and s2 a scale per column
+// (tensors `mixer_scale` and `feed_forward_scale`, [hidden]; empty names: none).  With `token_dim` n >= 1 an input of the token's own
+// follows: e = columns [token_offset, token_offset + n) of the token's row in the table that the model keeps beside its embedding,
+//   g = gelu_tanh(W_gate h) * e,   h += rmsnorm(W_proj g) * w      (tensors `<token>.gate` [n, hidden], `<token>.proj` [hidden, n],
+//                                                                   `<token>.norm` [hidden], eps inside the root)
+// The sums, the scales and the norms are float32.  The sum of both sublayers is one kernel, which takes the weighted sum of two mixers side
+// by side along; the token's part stays pending with its norm and rides in the next layer's norm (or the model's final one).
+class SharedNormBlock : public Arrangement {
+public:
+    struct Names { std::string mixer_scale, ff_scale, token; };
+    SharedNormBlock(const BlockParts& p, int hidden, double eps, const Names& names, bool feed_forward, int token_dim, int token_offset)
+        : p_(p), hidden_(hidden), eps_(static_cast<float>(eps)), names_(names), feed_forward_(feed_forward), n_(token_dim), offset_(token_offset) {
+        if (hidden <= 0) throw ConfigError("arrangement 'shared_norm': argument 'hidden' must be positive");
+        if (n_ < 0 || offset_ < 0) throw ConfigError("arrangement 'shared_norm': token_dim and token_offset must not be negative");
+    }
+    bool graph_safe() const override { return true; }
+
+    WeightTable weight_specs() const override {
+        WeightTable t;
+        for (const std::string& s : {names_.mixer_scale, feed_forward_ ? names_.ff_scale : std::string()}) {
+            if (s.empty()) continue;
+            t[s].shape = {hidden_};
+            t[s].init_ones = true;
+        }
+        if (n_ > 0) {
+            t[names_.token + ".gate"].shape = {n_, hidden_};
+            t[names_.token + ".proj"].shape = {hidden_, n_};
+            t[names_.token + ".norm"].shape = {hidden_};
+            t[names_.token + ".norm"].init_ones = true;
+        }
+        return t;
+    }
+    void bind(const Weights& w, BindContext& bc) override {
+        if (!names_.mixer_scale.empty()) scale_[0] = bc.upload(w.at(names_.mixer_scale), DType::F32);
+        if (feed_forward_ && !names_.ff_scale.empty()) scale_[1] = bc.upload(w.at(names_.ff_scale), DType::F32);
+        if (n_ == 0) return;
+        gate_.bind({&w.at(names_.token + ".gate")}, bc, 8);
+        proj_.bind({&w.at(names_.token + ".proj")}, bc);
+        norm_ = bc.upload(w.at(names_.token + ".norm"), DType::F32);
+    }
+
+    void* forward(StepContext& ctx, float* h, void* pending) override {
+        if (ctx.hidden != hidden_) throw ConfigError("arrangement 'shared_norm': the stream's width is not the one it was built for");
+        void* x = ctx.take_tokens(hidden_, ctx.act_dtype);
+        read_stream(ctx, h, pending, x);
+        void* y1 = ctx.take_tokens(hidden_, ctx.act_dtype);
+        ctx.takes_two_terms = true;
+        ctx.second_term = nullptr;
+        ctx.first_weight = 1.f;
+        ctx.second_weight = 0.f;
+        p_.mixer->forward(ctx, x, y1);
+        void* second = ctx.second_term;
+        ctx.takes_two_terms = false;
+        ctx.second_term = nullptr;
+        void* y2 = nullptr;
+        if (feed_forward_) {
+            y2 = ctx.take_tokens(hidden_, ctx.act_dtype);
+            p_.feed_forward->forward(ctx, x, y2);
+        }
+        // (the token's input reads the new stream in the activation dtype; x is free again and takes that copy)
+        const bool copies = n_ > 0 && ctx.act_dtype != DType::F32;
+        ops::scaled_sum(h, y1, ctx.first_weight, second, ctx.second_weight, fp(scale_[0]), y2, fp(scale_[1]), copies ? x : nullptr, ctx);
+        ctx.give(y2);
+        ctx.give(second);
+        ctx.give(y1);
+        void* left = n_ > 0 ? token_input(ctx, copies ? x : h) : nullptr;
+        ctx.give(x);
+        return left;
+    }
+
+private:
+    static const float* fp(const DeviceTensor& t) { return static_cast<const float*>(t.ptr); }
+
+    // x = norm(h), after what an earlier layer left pending has joined the stream
+    void read_stream(StepContext& ctx, float* h, void* pending, void* x) {
+        const float* nw = nullptr;
+        float eps = 0.f;
+        if (pending && ctx.pending_norm_weight && p_.mixer_norm->as_rms(&nw, &eps)) {
+            ops::norm_sum_norm(h, pending, nullptr, ctx.pending_norm_weight, ctx.pending_norm_eps, nw, eps, x, nullptr, ctx.T, hidden_, ctx.act_dtype, ctx.stream);
+            ctx.pending_norm_weight = nullptr;
+            ctx.give(pending);
+            return;
+        }
+        if (ctx.pending_norm_weight) {
+            settle_pending(ctx, h, pending, hidden_);
+            pending = nullptr;
+        }
+        p_.mixer_norm->forward(ctx, h, pending, x, nullptr, 0);
+        ctx.give(pending);
+    }
+
+    // W_proj (gelu(W_gate x) * e), left pending with its norm
+    void* token_input(StepContext& ctx, const void* x) {
+        if (!ctx.token_rows || ctx.token_rows->cols() < offset_ + n_)
+            throw ConfigError("arrangement 'shared_norm': the model's embedding keeps no rows per token that are wide enough for this layer");
+        const int ld = static_cast<int>(gate_.out_features);
+        float* z = static_cast<float*>(ctx.take_tokens(ld, DType::F32));
+        project_f32(ctx, gate_, x, z);
+        void* g = ctx.take_tokens(n_, ctx.act_dtype);
+        ops::gated_token_rows(z, ld, *ctx.token_rows, offset_, n_, g, ctx);
+        ctx.give(z);
+        void* y = ctx.take_tokens(hidden_, ctx.act_dtype);
+        project(ctx, proj_, g, y);
+        ctx.give(g);
+        ctx.pending_norm_weight = fp(norm_);
+        ctx.pending_norm_eps = eps_;
+        return y;
+    }
+
+    BlockParts p_;
+    int hidden_;
+    float eps_;
+    Names names_;
+    bool feed_forward_;
+    int n_, offset_;
+    DeviceTensor scale_[2], norm_;
+    Linear gate_, proj_;
+};
+
 // The feed-forward of a layer that has none: no weights, never run.
 class NoFeedForward : public FeedForward {
 public:
@@ -371,6 +490,17 @@ struct Reg {
             return std::make_shared<BothNormsBlock>(parts, static_cast<int>(arg_int(a, "hidden", k)), arg_number(a, "eps", k), arg_number_or(a, "share", 1.0, k),
                                                     arg_string_or(a, "mixer_out", "norm1b", k), arg_string_or(a, "feed_forward_out", "norm2b", k),
                                                     arg_int_or(a, "feed_forward", 1, k) != 0);
+        });
+        // one norm in front of both sublayers, which run side by side; an optional input of the token's own behind them
+        register_arrangement("shared_norm", [](const json::Value& a, const BlockParts& parts) {
+            const char* k = "shared_norm";
+            SharedNormBlock::Names n;
+            n.mixer_scale = arg_string_or(a, "mixer_scale", "", k);
+            n.ff_scale = arg_string_or(a, "feed_forward_scale", "", k);
+            n.token = arg_string_or(a, "token", "token", k);
+            return std::make_shared<SharedNormBlock>(parts, static_cast<int>(arg_int(a, "hidden", k)), arg_number(a, "eps", k), n,
+                                                     arg_int_or(a, "feed_forward", 1, k) != 0, static_cast<int>(arg_int_or(a, "token_dim", 0, k)),
+                                                     static_cast<int>(arg_int_or(a, "token_offset", 0, k)));
         });
         register_part("feed_forward", "none", [](const json::Value&) { return std::make_shared<NoFeedForward>(); });
     }

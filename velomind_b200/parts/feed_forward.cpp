@@ -9,11 +9,16 @@ namespace vmb {
 //
 // `activation` (VM_ACT_*) and the three tensors' names are arguments; the weight-streaming kernels take the activation as an
 // argument, the tcgen05 epilogue knows SiLU (other activations take the library products there).
+// With a positive `limit` the unit is the clamped one, not act(g) u: g <- min(g, limit), u <- clamp(u, -limit, limit),
+// g sigmoid(alpha g) (u + 1).
 class SwiGLU : public FeedForward {
 public:
     SwiGLU(int hidden, int intermediate, int activation = VM_ACT_SILU, std::string gate = "gate_proj.weight", std::string up = "up_proj.weight",
-           std::string down = "down_proj.weight")
-        : hidden_(hidden), I_(intermediate), act_(activation), gate_name_(std::move(gate)), up_name_(std::move(up)), down_name_(std::move(down)) {}
+           std::string down = "down_proj.weight", float limit = 0.f, float alpha = 1.702f)
+        : hidden_(hidden), I_(intermediate), act_(activation), gate_name_(std::move(gate)), up_name_(std::move(up)), down_name_(std::move(down)), limit_(limit),
+          alpha_(alpha) {
+        if (limit_ < 0.f) throw ConfigError("part 'gated': limit must not be negative");
+    }
 
     WeightTable weight_specs() const override {
         WeightTable t;
@@ -50,7 +55,7 @@ public:
         float eps = 0.f;
         norm.as_rms(&nw, &eps);
         const bool skinny = ctx.T_cap <= max_rows();
-        const bool tc = !skinny && act_ == VM_ACT_SILU && ops::tc_fused_rows(ctx) && I_ % 64 == 0;      // (that epilogue knows SiLU)
+        const bool tc = !skinny && act_ == VM_ACT_SILU && !clamped() && ops::tc_fused_rows(ctx) && I_ % 64 == 0;      // (that epilogue knows SiLU)
         if (!skinny && !tc) {
             // the library's products: norm, gate and up, SwiGLU, down added into h by the product itself
             void* x = ctx.take_tokens(hidden_, DType::BF16);
@@ -59,7 +64,7 @@ public:
             ops::linear(x, DType::BF16, hidden_, gate_up_.weight, gu, DType::BF16, ctx.T, ctx.stream);
             ctx.give(x);
             void* a = ctx.take_tokens(I_, DType::BF16);
-            ops::gated_activation(gu, a, ctx.T, I_, act_, DType::BF16, ctx.stream);
+            unit(ctx, gu, a);
             ctx.give(gu);
             ops::linear_residual(a, I_, down_.weight, h, ctx.T, ctx.stream);
             ctx.give(a);
@@ -67,11 +72,11 @@ public:
         }
         void* act = ctx.take_tokens(I_, DType::BF16);
         if (skinny && ctx.T_cap <= ops::SKINNY_NORM_ROWS) {
-            ops::skinny_gated(h, nw, eps, gate_up_.weight, ctx.T, I_, act_, act, ctx.err, ctx.stream);
+            few_rows(ctx, h, nw, eps, act);
         } else {
             void* x = ctx.take_tokens(hidden_, DType::BF16);           // many rows: norm once, not once per CTA
             norm.forward(ctx, h, nullptr, x, nullptr, 0);
-            if (skinny) ops::skinny_gated(x, nullptr, 0.f, gate_up_.weight, ctx.T, I_, act_, act, ctx.err, ctx.stream);
+            if (skinny) few_rows(ctx, x, nullptr, 0.f, act);
             else ops::tc_swiglu(x, hidden_, gate_up_.weight, ctx.T, I_, act, ctx.err, ctx.stream);
             ctx.give(x);
         }
@@ -85,7 +90,7 @@ public:
         if (ctx.act_dtype == DType::BF16 && gate_up_.weight.dtype == DType::BF16 && down_.weight.dtype == DType::BF16 && ctx.T_cap <= max_rows() &&
             hidden_ % 32 == 0 && I_ % 32 == 0 && ctx.T > 0) {
             void* act = ctx.take_tokens(I_, DType::BF16);
-            ops::skinny_gated(x, nullptr, 0.f, gate_up_.weight, ctx.T, I_, act_, act, ctx.err, ctx.stream);
+            few_rows(ctx, x, nullptr, 0.f, act);
             ops::skinny_linear(act, nullptr, 0.f, down_.weight, ctx.T, out, hidden_, false, nullptr, ctx.err, ctx.stream);
             ctx.give(act);
             return;
@@ -93,15 +98,26 @@ public:
         void* gu = ctx.take_tokens(2ll * I_, ctx.act_dtype);
         gate_up_.apply(ctx, x, ctx.act_dtype, gu, ctx.act_dtype, ctx.T, ctx.T_cap);
         void* act = ctx.take_tokens(I_, ctx.act_dtype);
-        ops::gated_activation(gu, act, ctx.T, I_, act_, ctx.act_dtype, ctx.stream);
+        unit(ctx, gu, act);
         ctx.give(gu);
         down_.apply(ctx, act, ctx.act_dtype, out, ctx.act_dtype, ctx.T, ctx.T_cap);
         ctx.give(act);
     }
 
 private:
+    bool clamped() const { return limit_ > 0.f; }
+    void unit(StepContext& ctx, const void* gu, void* out) {
+        if (clamped()) ops::clamped_unit(gu, out, ctx.T, I_, limit_, alpha_, ctx.act_dtype, ctx.stream);
+        else ops::gated_activation(gu, out, ctx.T, I_, act_, ctx.act_dtype, ctx.stream);
+    }
+    // few rows: both products and the unit in one kernel (nw given: of the norm of the float32 residual rows)
+    void few_rows(StepContext& ctx, const void* x, const float* nw, float eps, void* out) {
+        if (clamped()) ops::skinny_clamped(x, nw, eps, gate_up_.weight, ctx.T, I_, limit_, alpha_, out, ctx.err, ctx.stream);
+        else ops::skinny_gated(x, nw, eps, gate_up_.weight, ctx.T, I_, act_, out, ctx.err, ctx.stream);
+    }
     int hidden_, I_, act_;
     std::string gate_name_, up_name_, down_name_;
+    float limit_, alpha_;
     Linear gate_up_, down_;
 };
 
@@ -216,7 +232,8 @@ RegisterPart reg_gated("feed_forward", "gated", [](const json::Value& a) {
     const char* k = "gated";
     return std::make_shared<SwiGLU>(static_cast<int>(arg_int(a, "hidden", k)), static_cast<int>(arg_int(a, "intermediate", k)),
                                     activation_code(arg_string_or(a, "activation", "silu", k), k), arg_string_or(a, "gate", "gate_proj.weight", k),
-                                    arg_string_or(a, "up", "up_proj.weight", k), arg_string_or(a, "down", "down_proj.weight", k));
+                                    arg_string_or(a, "up", "up_proj.weight", k), arg_string_or(a, "down", "down_proj.weight", k),
+                                    static_cast<float>(arg_number_or(a, "limit", 0.0, k)), static_cast<float>(arg_number_or(a, "alpha", 1.702, k)));
 });
 // the unit without a gate
 RegisterPart reg_mlp("feed_forward", "mlp", [](const json::Value& a) {

@@ -9,6 +9,7 @@
 //   `unit_heads`: every q and k head divided by its root mean square over `dim` (a norm without a weight)
 //   `position`: rotary positions on the first rotary_dim values of every q and k head, either pairing
 //   score(i, j) = scale q_i . k_j;  i sees j  iff  j <= i and (window == 0 or i - j < window or j < keep_first)
+//   `chunk` C >= 1 instead of a window: i sees j iff j <= i and floor(i / C) = floor(j / C), chunks counted from the sequence's start
 //   `slopes`: 2^(-8 (h + 1) / H) (i - j) comes off head h's score of key j
 //   `own_kv` = 0: the layer has no k and v of its own; its schedule entry names the run whose keys and values (as cached) it reads, with its
 //       own queries, window and everything else
@@ -38,6 +39,7 @@ public:
         scale_ = static_cast<float>(arg_number_or(a, "scale", 1.0 / std::sqrt(static_cast<double>(Dk_)), k));
         window_ = static_cast<int>(arg_int_or(a, "window", 0, k));
         keep_first_ = static_cast<int>(arg_int_or(a, "keep_first", 0, k));
+        chunk_ = static_cast<int>(arg_int_or(a, "chunk", 0, k));
         K_ = static_cast<int>(arg_int_or(a, "taps", 0, k));
         bias_ = arg_int_or(a, "bias", 0, k) != 0;
         out_bias_ = arg_int_or(a, "out_bias", 0, k) != 0;
@@ -57,6 +59,7 @@ public:
         if (values_are_keys_ && Dv_ != Dk_) throw ConfigError(format("part '%s': values that are the keys have the keys' size (vdim %d, dim %d)", k, Dv_, Dk_));
         if (window_ < 0 || keep_first_ < 0) throw ConfigError(format("part '%s': window and keep_first must not be negative", k));
         if (window_ == 0) keep_first_ = 0;
+        if (chunk_ < 0 || (chunk_ > 0 && window_ > 0)) throw ConfigError(format("part '%s': chunk must not be negative and excludes a window", k));
         if (K_ < 0 || K_ > 16) throw ConfigError(format("part '%s': taps (%d) must be within 0..16", k, K_));
         if (qk_norm_ && unit_heads_) throw ConfigError(format("part '%s': qk_norm and unit_heads exclude each other", k));
         if (!own_ && (K_ >= 1 || values_are_keys_ || qk_norm_))
@@ -128,11 +131,12 @@ public:
 
     CacheNeed cache_need() const override {
         CacheNeed n;
-        n.kind = window_ > 0 ? CacheNeed::Window : CacheNeed::All;
+        n.kind = window_ > 0 ? CacheNeed::Window : (chunk_ > 0 ? CacheNeed::Chunk : CacheNeed::All);
         n.kv_heads = G_;
         n.key_dim = Dk_;
         n.value_dim = Dv_;
         n.window = window_;
+        n.chunk = chunk_;
         n.keep_first = keep_first_;
         n.state_floats = K_ > 1 ? static_cast<int>((K_ - 1) * row_cols()) : 0;
         return n;
@@ -164,6 +168,7 @@ public:
         void* att = ctx.take_tokens(static_cast<long long>(H_) * Dv_, act);
         ops::BiasedMask mask;
         mask.window = window_;
+        mask.chunk = chunk_;
         mask.keep_first = keep_first_;
         mask.sink = sink_ ? static_cast<const float*>(sinks_.ptr) : nullptr;
         mask.slopes = slopes_ ? static_cast<const float*>(slope_.ptr) : nullptr;
@@ -179,7 +184,7 @@ public:
     }
 
 private:
-    int hidden_ = 0, H_ = 0, G_ = 0, Dk_ = 0, Dv_ = 0, window_ = 0, keep_first_ = 0, K_ = 0, gate_cols_ = 0, gate_per_ = 1;
+    int hidden_ = 0, H_ = 0, G_ = 0, Dk_ = 0, Dv_ = 0, window_ = 0, keep_first_ = 0, chunk_ = 0, K_ = 0, gate_cols_ = 0, gate_per_ = 1;
     float scale_ = 1.f, eps_ = 1e-6f;
     bool bias_ = false, out_bias_ = false, qk_norm_ = false, sink_ = false, values_are_keys_ = false, unit_heads_ = false, slopes_ = false, own_ = true;
     std::shared_ptr<Position> position_;

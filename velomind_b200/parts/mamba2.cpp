@@ -113,11 +113,11 @@ public:
 
     void forward(StepContext& ctx, const void* x, void* out) override {
         void* proj = ctx.take_tokens(width(), ctx.act_dtype);
-        in_.apply(ctx, x, ctx.act_dtype, proj, ctx.act_dtype, ctx.T, ctx.T_cap);
+        project(ctx, in_, x, proj);
         void* y = ctx.take_tokens(inner(), ctx.act_dtype);
         mix(ctx, proj, y);
         ctx.give(proj);
-        out_.apply(ctx, y, ctx.act_dtype, out, ctx.act_dtype, ctx.T, ctx.T_cap);
+        project(ctx, out_, y, out);
         ctx.give(y);
     }
 

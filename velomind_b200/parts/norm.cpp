@@ -9,14 +9,19 @@ namespace vmb {
 class RMSNorm : public Norm {
 public:
     // `tensor`: what the scale is called behind the part's prefix ("weight" unless the checkpoint says otherwise; may be empty)
-    RMSNorm(int size, float eps, std::string tensor = "weight") : size_(size), eps_(eps), tensor_(std::move(tensor)) {}
+    // `about_one`: the tensor holds the scale's distance from 1; the sum is made once, in float32, when the weight is bound
+    RMSNorm(int size, float eps, std::string tensor = "weight", bool about_one = false)
+        : size_(size), eps_(eps), tensor_(std::move(tensor)), about_one_(about_one) {}
     WeightTable weight_specs() const override {
         WeightSpec s;
         s.shape = {size_};
-        s.init_ones = true;
+        s.init_ones = !about_one_;
         return {{tensor_, s}};
     }
-    void bind(const Weights& w, BindContext& bc) override { weight_ = bc.upload(w.at(tensor_), DType::F32); }   // exact for BF16 and F32 storage
+    void bind(const Weights& w, BindContext& bc) override {
+        if (about_one_) weight_ = bc.upload_mapped(w.at(tensor_), [](float v) { return 1.0f + v; });
+        else weight_ = bc.upload(w.at(tensor_), DType::F32);       // exact for BF16 and F32 storage
+    }
     bool graph_safe() const override { return true; }
     bool as_rms(const float** weight, float* eps) const override {
         *weight = static_cast<const float*>(weight_.ptr);
@@ -31,13 +36,14 @@ private:
     int size_;
     float eps_;
     std::string tensor_;
+    bool about_one_;
     DeviceTensor weight_;
 };
 
 namespace {
 RegisterPart reg("norm", "rmsnorm", [](const json::Value& a) {
     return std::make_shared<RMSNorm>(static_cast<int>(arg_int(a, "size", "rmsnorm")), static_cast<float>(arg_number(a, "eps", "rmsnorm")),
-                                     arg_string_or(a, "tensor", "weight", "rmsnorm"));
+                                     arg_string_or(a, "tensor", "weight", "rmsnorm"), arg_int_or(a, "about_one", 0, "rmsnorm") != 0);
 });
 
 // The norm of a layer half that does not exist (a layer without a feed-forward): no weights, never run.

@@ -17,7 +17,7 @@
 // scores are the weights, not renormalised; there is no correction tensor unless `correction` = 1.  A third form of expert (`glu` = 2):
 // W_down (silu(W_gate h) * (W_up h)) where the routing weight multiplies the expert's INPUT, h = w x, not its output; the shared expert
 // (tensors shared.gate, shared.up, shared.down) has the same form and runs with w = 1, without a gate of its own.  `glu` = 3 is the same unit
-// with the routing weight on the expert's OUTPUT.  `groups_top` = n makes a group's score the sum of its n largest scores (default 1).
+// with the routing weight on the expert's OUTPUT.  `normalize` = 1 (of the scored forms): the weights are the chosen scores over their sum.  `groups_top` = n makes a group's score the sum of its n largest scores (default 1).
 #include "args.h"
 #include "linear.h"
 
@@ -39,6 +39,7 @@ struct Routing {
     float limit = 0.f, alpha = 1.702f;
     int score_kind = VM_SCORE_SOFTMAX;   // of the scored form
     bool correction = true;              // the scored form has a correction tensor
+    bool normalize = false;              // of the scored form: the chosen scores are divided by their sum (+ 1e-20)
 };
 
 class RoutedExperts : public FeedForward {
@@ -148,7 +149,7 @@ public:
         if (r_.scored) {
             if (gate_) throw Error("routed_experts: the scored router has no gate for a shared expert");
             ops::expert_router_scored(x, nw, eps, static_cast<const float*>(router_.ptr), r_.correction ? static_cast<const float*>(router_b_.ptr) : nullptr,
-                                      ctx.T, hidden_, E_ + r_.identity, top_, r_.groups, r_.groups_keep, r_.groups_top, r_.scale, r_.score_kind, chosen, weight,
+                                      ctx.T, hidden_, E_ + r_.identity, top_, r_.groups, r_.groups_keep, r_.groups_top, r_.scale, r_.score_kind, r_.normalize, chosen, weight,
                                       ctx.act_dtype, ctx.stream);
             return;
         }
@@ -267,6 +268,8 @@ RegisterPart reg("feed_forward", "routed_experts", [](const json::Value& a) {
     r.groups_top = static_cast<int>(arg_int_or(a, "groups_top", 1, k));
     r.identity = static_cast<int>(arg_int_or(a, "identity", 0, k));
     r.scale = static_cast<float>(arg_number_or(a, "scale", 1.0, k));
+    r.normalize = arg_int_or(a, "normalize", 0, k) != 0;
+    if (r.normalize && !r.scored) throw ConfigError("part 'routed_experts': normalize belongs to the scored forms of routing");
     r.glu = static_cast<int>(arg_int_or(a, "glu", 0, k));
     if (r.glu < VM_GLU_NONE || r.glu > VM_GLU_SILU) throw ConfigError("part 'routed_experts': glu is 0 (none), 1 (clamped), 2 (SiLU, weight on the input) or 3 (SiLU, weight on the output)");
     r.limit = static_cast<float>(arg_number_or(a, "limit", 0.0, k));

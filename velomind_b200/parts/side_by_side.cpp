@@ -65,14 +65,22 @@ public:
     }
 
     void forward(StepContext& ctx, const void* x, void* out) override {
+        const bool leaves = !normed_ && ctx.takes_two_terms;      // the wiring carries the weighted sum out
+        ctx.takes_two_terms = false;
         ctx.takes_row_bias = false;                       // (two results are joined first: neither may leave its bias to the wiring)
         const int base = ctx.state_offset;
-        void* a = ctx.take_tokens(hidden_, ctx.act_dtype);
+        void* a = leaves ? out : ctx.take_tokens(hidden_, ctx.act_dtype);
         left_->forward(ctx, x, a);
         ctx.state_offset = base + left_->cache_need().state_floats;
         void* b = ctx.take_tokens(hidden_, ctx.act_dtype);
         right_->forward(ctx, x, b);
         ctx.state_offset = base;
+        if (leaves) {
+            ctx.second_term = b;
+            ctx.first_weight = left_scale_;
+            ctx.second_weight = right_scale_;
+            return;
+        }
         ops::join_rows(a, b, nullptr, left_scale_, right_scale_, normed_ ? static_cast<const float*>(wl_.ptr) : nullptr,
                        normed_ ? static_cast<const float*>(wr_.ptr) : nullptr, eps_, out, ctx.T, hidden_, ctx.act_dtype, ctx.stream);
         ctx.give(b);
