@@ -367,6 +367,34 @@ def zabozen_config(z, x):
                        {"type": "attention", "mixer": dict(att, mask={"size": x["reader_window"]}, kv_from=0), "mlp": dense}]}
 
 
+# ------------------------------------------------------------------------------------------------ --design depunex
+# The same widths, four layers with one norm for both sublayers and an input of the token's own: Mamba-2 + clamped gated unit; chunked
+# attention beside the selective scan + routed experts; Mamba-2 + routed experts; the second layer's mixer + clamped gated unit.  Beside it
+# Semesun (the same Mamba-2 sizes, windowed attention with the same kernels, routed experts in groups), Vozetar (two mixers side by side,
+# the same pair table) and the Llama decoder at equal width and depth.
+DEPUNEX_EXTRA = {
+    "w1024": dict(kv_heads=4, chunk=1024, ssm_heads=32, ssm_vdim=64, ssm_state=128, ssm_groups=1, inner=2048, dt_rank=64, scan_state=16, token_dim=128,
+                  groups=2, keep=1),
+    "w2048": dict(kv_heads=8, chunk=1024, ssm_heads=64, ssm_vdim=64, ssm_state=128, ssm_groups=1, inner=4096, dt_rank=128, scan_state=16, token_dim=256,
+                  groups=2, keep=1),
+}
+
+
+def depunex_config(z, x):
+    att = {"heads": z["heads"], "kv_heads": x["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5, "mask": {"size": x["chunk"]},
+           "rot": {"base": 500000.0, "dims": z["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    scan = {"inner": x["inner"], "dt_rank": x["dt_rank"], "state": x["scan_state"], "conv": 4}
+    par = {"left": att, "left_scale": 0.7, "right": scan, "right_scale": 0.7}
+    ssm = {"heads": x["ssm_heads"], "vdim": x["ssm_vdim"], "state": x["ssm_state"], "groups": x["ssm_groups"], "conv": 4, "norm_groups": 1}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": x["groups"], "keep": x["keep"]}}}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    return {"architecture": "Depunex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "token_side": {"dim": x["token_dim"]},
+            "embedding": {"scale": z["width"] ** 0.5, "bigram": {"buckets": 100003, "mul_prev": 8191, "mul_cur": 31}},
+            "layers": [{"type": "mamba2", "mixer": ssm, "mlp": dense}, {"type": "parallel", "mixer": par, "mlp": moe},
+                       {"type": "mamba2", "mixer": ssm, "mlp": moe}, {"type": "parallel", "mixer": par, "mlp": dense}]}
+
+
 def kogilix_attention_config(z):
     att = {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"], "scale": z["dim"] ** -0.5}
     moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["shared_ff"]}}
@@ -395,7 +423,7 @@ def op_table(vm, engine, entries):
 
 
 def design_arm(args):
-    """Prompt and decode throughput of a design (Kogilix, Semesun, Fidizen, Vozetar, Zabozen) at a few sizes, beside the library's other models at equal size."""
+    """Prompt and decode throughput of a design (Kogilix, Semesun, Fidizen, Vozetar, Zabozen, Depunex) at a few sizes, beside the library's other models at equal size."""
     import numpy as np
     import velomind_b200 as vm
     T, B, prompt_len = 2048, 8, 512
@@ -412,6 +440,9 @@ def design_arm(args):
             models = [("vozetar", vozetar_config(z, VOZETAR_EXTRA[name])), ("semesun", semesun_config(z, SEMESUN_EXTRA[name])), ("llama", llama_config_like(z))]
         if args.design == "zabozen":
             models = [("zabozen", zabozen_config(z, ZABOZEN_EXTRA[name])), ("fidizen", fidizen_config(z, FIDIZEN_EXTRA[name])),
+                      ("vozetar", vozetar_config(z, VOZETAR_EXTRA[name])), ("llama", llama_config_like(z))]
+        if args.design == "depunex":
+            models = [("depunex", depunex_config(z, DEPUNEX_EXTRA[name])), ("semesun", semesun_config(z, SEMESUN_EXTRA[name])),
                       ("vozetar", vozetar_config(z, VOZETAR_EXTRA[name])), ("llama", llama_config_like(z))]
         if args.design == "fidizen":
             models = [("fidizen", fidizen_config(z, FIDIZEN_EXTRA[name])), ("kogilix_attention", kogilix_attention_config(z)), ("llama", llama_config_like(z))]
@@ -543,7 +574,7 @@ def main() -> int:
     ap.add_argument("--quick", action="store_true", help="skip the batch 1 / 64 points and the end-to-end run")
     ap.add_argument("--shape", default="135m", choices=sorted(SHAPES),
                     help="sizes of the random model: the benchmark's SmolLM2-135M (default), or the 360M / 1.7B shapes of the family")
-    ap.add_argument("--design", default="", choices=["", "kogilix", "semesun", "fidizen", "vozetar", "zabozen"],
+    ap.add_argument("--design", default="", choices=["", "kogilix", "semesun", "fidizen", "vozetar", "zabozen", "depunex"],
                     help="instead of the benchmark: prompt and decode throughput of another design of the library at a few layer sizes, "
                          "beside the Llama decoder at equal size (one JSON line of its own)")
     args = ap.parse_args()

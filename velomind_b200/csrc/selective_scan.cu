@@ -12,11 +12,11 @@
 // Four lanes (a quad) share a channel; lane q of the quad holds the states n = 4 V (i / V) + V q + i % V, V of them side by side, so that
 // the quad's reads of B and C from shared memory lie side by side.
 //
-// Prompts.  Tokens are taken four at a time.  Lane q works out token q's step size for the quad, hands it round, and, after the four sums
-// of y are exchanged (each lane ends up with one token's), finishes token q's output.  One pass over the tokens suffices where a step has
-// enough channels and sequences; else the tokens are cut into pieces that run side by side: a first pass leaves what every piece adds to
-// the state and the sum of its step sizes, a second one carries the state from piece to piece, a third one repeats the pieces from the right
-// start.
+// Prompts.  Tokens come through shared memory sixteen at a time, asked for several stages ahead.  A block first works out the step sizes of
+// the next sixteen (each thread four of them), then runs the recurrence over the current sixteen without a branch or a barrier; after every
+// four tokens the quad exchanges its partial sums of y so that each lane ends up with one token's, and finishes those outputs at the end.  One pass over the tokens suffices where a step has enough channels and
+// sequences; else the tokens are cut into pieces that run side by side: a first pass leaves what every piece adds to the state and the sum of
+// its step sizes, a second one carries the state from piece to piece, a third one repeats the pieces from the right start.
 //
 // Decode steps.  One launch: the step size's dot product, the state's update and the gated output.
 #include "short_conv.cuh"
@@ -25,12 +25,30 @@ namespace {
 
 constexpr int SS_THREADS = 64;                 // 16 channels
 constexpr int SS_CH = SS_THREADS / 4;
+constexpr int SS_TT = 16;                      // tokens per stage
+constexpr int SS_STAGES = 4;                   // stages of shared memory: a stage's rows are asked for 48 tokens ahead
 
 __device__ __forceinline__ float ss_exp2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+
+// log(1 + e^z) = max(z, 0) + log1p(e^-|z|) without a branch: with u = e^-|z| in (0, 1] and w = u / (2 + u) <= 1/3,
+// log1p(u) = 2 atanh(w) = 2 (w + w^3 / 3 + w^5 / 5 + ...); seven terms leave less than 1e-8 of the sum.
+__device__ __forceinline__ float ss_softplus(float z) {
+    const float u = expf(-fabsf(z));
+    const float w = __fdividef(u, 2.0f + u), w2 = w * w;
+    float a = fmaf(w2, 1.0f / 13.0f, 1.0f / 11.0f);
+    a = fmaf(w2, a, 1.0f / 9.0f);
+    a = fmaf(w2, a, 1.0f / 7.0f);
+    a = fmaf(w2, a, 1.0f / 5.0f);
+    a = fmaf(w2, a, 1.0f / 3.0f);
+    a = fmaf(w2, a, 1.0f);
+    return fmaf(2.0f * w, a, fmaxf(z, 0.0f));
+}
+// z sigmoid(z) without a branch
+__device__ __forceinline__ float ss_silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 
 // states of lane q: index i -> n
 template <int V> __device__ __forceinline__ int ss_state_of(int q, int i) { return (i / V) * 4 * V + q * V + i % V; }
@@ -44,6 +62,13 @@ template <> __device__ __forceinline__ void ss_load<4>(const float* p, float* v)
 template <> __device__ __forceinline__ void ss_load<2>(const float* p, float* v) {
     const float2 f = *reinterpret_cast<const float2*>(p);
     v[0] = f.x; v[1] = f.y;
+}
+
+// 16 bytes to shared memory (zeros where there is nothing to read)
+__device__ __forceinline__ void ss_copy16(void* smem, const void* gmem, bool in) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(smem);
+    const int bytes = in ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(gmem), "r"(bytes));
 }
 
 // the piece a block works on: sequence, first token, tokens.  Pieces are cut at multiples of `piece` new tokens of their sequence.
@@ -70,77 +95,131 @@ struct ScanParams {
     const int *cu_tokens, *slots;
     void* out;                  // [T, C] (activation dtype)
     int ldt, ldr, b_col, ldz, B, C, N, piece;
+    int vec;                    // rows may be copied 16 bytes at a time
 };
 
 enum { SS_WHOLE = 0, SS_ADDS = 1, SS_FROM_START = 2 };
+
+template <typename T, int NPT> constexpr int ss_stage_bytes() { return SS_TT * (2 * 4 * NPT * 4 + SS_CH * 4 + 2 * SS_CH * (int)sizeof(T)); }
 
 template <typename T, int NPT, int MODE>
 __global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(const ScanParams p) {
     constexpr int V = NPT % 4 == 0 ? 4 : 2;
     constexpr int NP = 4 * NPT;                               // states with padding
-    constexpr int SS_TT = NPT >= 32 ? 16 : 32;                // tokens of B and C in shared memory at a time
-    __shared__ __align__(16) float sBC[2][SS_TT][2 * NP];
+    constexpr int STAGE = ss_stage_bytes<T, NPT>();
+    __shared__ float2 sdt[2][SS_TT * SS_CH];                  // (dt, dt x)
+    extern __shared__ __align__(16) unsigned char ss_smem[];  // per stage: B | C [TT][2 NP], dt [TT][CH], x [TT][CH], z [TT][CH]
     int seq, t0, len;
     if (!ss_where(p.cu_tokens, p.B, p.piece, blockIdx.y, seq, t0, len)) return;
-    const int tid = threadIdx.x, q = tid & 3;
-    const int c = blockIdx.x * SS_CH + (tid >> 2);
+    const int tid = threadIdx.x, q = tid & 3, ch = tid >> 2;
+    const int c0 = blockIdx.x * SS_CH, c = c0 + ch;
     const bool live = c < p.C;
-    const int cc = live ? c : p.C - 1;                        // (idle quads follow the last channel and store nothing)
+    const int cc = live ? c : p.C - 1;                        // (idle quads store nothing)
+    auto at = [&](int stage) { return ss_smem + (size_t)(stage % SS_STAGES) * STAGE; };
+    if (NP > p.N)                                             // padded states read zeros
+        for (int i = tid; i < SS_STAGES * SS_TT * 2 * NP; i += SS_THREADS) {
+            const int row = i / (2 * NP), col = i - row * 2 * NP;
+            if (col % NP >= p.N) reinterpret_cast<float*>(at(row / SS_TT))[(row % SS_TT) * 2 * NP + col] = 0.f;
+        }
+    // tokens [base, base + TT) of the piece into a stage
+    auto load = [&](int base) {
+        unsigned char* sm = at(base / SS_TT);
+        float* bc = reinterpret_cast<float*>(sm);
+        float* dts = bc + SS_TT * 2 * NP;
+        T* xs = reinterpret_cast<T*>(dts + SS_TT * SS_CH);
+        T* zs = xs + SS_TT * SS_CH;
+        constexpr int E = 16 / (int)sizeof(T);                // values per 16 bytes
+        constexpr int WIDE = MODE == SS_ADDS ? 1 : 2;
+        if (p.vec) {
+#pragma unroll
+            for (int i = tid; i < SS_TT * WIDE * NPT; i += SS_THREADS) {      // (a padded row of B or C has NPT runs of four)
+                const int k = i / (WIDE * NPT), j = i - k * WIDE * NPT, half = j / NPT, n = 4 * (j - half * NPT);
+                const bool in = base + k < len;
+                if (n < p.N) ss_copy16(bc + k * 2 * NP + half * NP + n, p.r + (size_t)(t0 + (in ? base + k : 0)) * p.ldr + p.b_col + half * p.N + n, in);
+            }
+#pragma unroll
+            for (int i = tid; i < SS_TT * (SS_CH / 4); i += SS_THREADS) {
+                const int k = i / (SS_CH / 4), j = 4 * (i - k * (SS_CH / 4));
+                const bool in = base + k < len && c0 + j < p.C;
+                ss_copy16(dts + k * SS_CH + j, p.dt + (size_t)(t0 + (in ? base + k : 0)) * p.ldt + (in ? c0 + j : 0), in);
+            }
+#pragma unroll
+            for (int i = tid; i < SS_TT * (SS_CH / E); i += SS_THREADS) {
+                const int k = i / (SS_CH / E), j = E * (i - k * (SS_CH / E));
+                const bool in = base + k < len && c0 + j < p.C;
+                const size_t row = (size_t)(t0 + (in ? base + k : 0));
+                ss_copy16(xs + k * SS_CH + j, static_cast<const T*>(p.x) + row * p.C + (in ? c0 + j : 0), in);
+                if (MODE != SS_ADDS) ss_copy16(zs + k * SS_CH + j, static_cast<const T*>(p.z) + row * p.ldz + (in ? c0 + j : 0), in);
+            }
+            return;
+        }
+        for (int i = tid; i < SS_TT * 2 * p.N; i += SS_THREADS) {
+            const int k = i / (2 * p.N), j = i - k * 2 * p.N, half = j >= p.N, n = j - half * p.N;
+            bc[k * 2 * NP + half * NP + n] = base + k < len ? p.r[(size_t)(t0 + base + k) * p.ldr + p.b_col + half * p.N + n] : 0.f;
+        }
+        for (int i = tid; i < SS_TT * SS_CH; i += SS_THREADS) {
+            const int k = i / SS_CH, j = i - k * SS_CH;
+            const bool in = base + k < len && c0 + j < p.C;
+            const size_t row = (size_t)(t0 + base + k);
+            dts[i] = in ? p.dt[row * p.ldt + c0 + j] : 0.f;
+            xs[i] = in ? static_cast<const T*>(p.x)[row * p.C + c0 + j] : vm_from_float<T>(0.f);
+            zs[i] = in && MODE != SS_ADDS ? static_cast<const T*>(p.z)[row * p.ldz + c0 + j] : vm_from_float<T>(0.f);
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < SS_STAGES - 1; ++k) {
+        if (k * SS_TT < len) load(k * SS_TT);
+        asm volatile("cp.async.commit_group;\n" ::);
+    }
     float A2[NPT], s[NPT];
     float* S = p.state + (size_t)p.slots[seq] * p.state_stride + (size_t)cc * p.N;
     float* piece_S = MODE == SS_WHOLE ? nullptr : p.pieces + ((size_t)blockIdx.y * p.C + cc) * p.N;
+    const float* start = MODE == SS_WHOLE ? S : (MODE == SS_FROM_START ? piece_S : nullptr);
 #pragma unroll
     for (int i = 0; i < NPT; ++i) {
         const int n = ss_state_of<V>(q, i);
         A2[i] = n < p.N ? p.A2[(size_t)cc * p.N + n] : 0.f;
-        s[i] = 0.f;
-        if (MODE == SS_WHOLE && n < p.N) s[i] = S[n];
-        if (MODE == SS_FROM_START && n < p.N) s[i] = piece_S[n];
+        s[i] = start && n < p.N ? start[n] : 0.f;
     }
-    const float bias = p.dt_bias[cc], skip = MODE == SS_ADDS ? 0.f : p.D[cc];
+    const float skip = MODE == SS_ADDS ? 0.f : p.D[cc];
     float dt_sum = 0.f;
-    const T* xg = static_cast<const T*>(p.x) + cc;
-    const T* zg = static_cast<const T*>(p.z) + cc;
-    const float* dtg = p.dt + cc;
     T* og = static_cast<T*>(p.out) + cc;
 
-    auto stage = [&](int base, int buf) {                     // B and C of tokens [base, base + SS_TT) of the piece
-        for (int i = tid; i < SS_TT * 2 * NP; i += SS_THREADS) {
-            const int k = i / (2 * NP), col = i - k * 2 * NP;
-            const int n = col < NP ? col : col - NP;
-            float v = 0.f;
-            if (base + k < len && n < p.N) v = p.r[(size_t)(t0 + base + k) * p.ldr + p.b_col + (col < NP ? 0 : p.N) + n];
-            sBC[buf][k][col] = v;
+    // step sizes of a stage's tokens for the block's channels; 0 past the end (the state then stays as it is)
+    const int my_ch = tid & (SS_CH - 1), my_c = min(c0 + my_ch, p.C - 1);
+    const float bias = p.dt_bias[my_c];
+    auto steps = [&](int base) {
+        const float* bc = reinterpret_cast<const float*>(at(base / SS_TT));
+        const float* dts = bc + SS_TT * 2 * NP;
+        const T* xs = reinterpret_cast<const T*>(dts + SS_TT * SS_CH);
+        float2* out = sdt[(base / SS_TT) & 1];
+#pragma unroll
+        for (int j = 0; j < SS_TT * SS_CH / SS_THREADS; ++j) {
+            const int k = (tid + j * SS_THREADS) / SS_CH;
+            const float dt = base + k < len ? ss_softplus(dts[k * SS_CH + my_ch] + bias) : 0.f;
+            out[k * SS_CH + my_ch] = make_float2(dt, dt * vm_to_float(xs[k * SS_CH + my_ch]));
         }
     };
-    // lane q's own token of a group of four: raw step size, input, gate
-    float n_dt, n_x, n_z;
-    auto fetch = [&](int g) {
-        const int t = g + q;
-        const bool in = t < len;
-        const size_t row = (size_t)(t0 + (in ? t : len - 1));
-        n_dt = dtg[row * p.ldt];
-        n_x = vm_to_float(xg[row * p.C]);
-        n_z = MODE == SS_ADDS ? 0.f : vm_to_float(zg[row * p.ldz]);
-    };
-    stage(0, 0);
-    fetch(0);
+    asm volatile("cp.async.wait_group %0;\n" ::"n"(SS_STAGES - 2));
     __syncthreads();
+    steps(0);
     for (int base = 0; base < len; base += SS_TT) {
-        const int buf = (base / SS_TT) & 1;
-        if (base + SS_TT < len) stage(base + SS_TT, buf ^ 1);
-        const int cnt = min(SS_TT, len - base);
-        for (int g = 0; g < cnt; g += 4) {
-            const bool in = base + g + q < len;
-            const float my_dt = in ? softplus_f(n_dt + bias) : 0.f;      // a token past the end: the state stays as it is
-            const float my_x = n_x, my_z = n_z, my_dx = my_dt * my_x;
-            if (base + g + 4 < len) fetch(base + g + 4);
-            if (MODE == SS_ADDS) dt_sum += my_dt;
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(SS_STAGES - 3));
+        __syncthreads();                                      // the next stage and this one's step sizes are there; the stage before is read by all
+        if (base + (SS_STAGES - 1) * SS_TT < len) load(base + (SS_STAGES - 1) * SS_TT);
+        asm volatile("cp.async.commit_group;\n" ::);
+        if (base + SS_TT < len) steps(base + SS_TT);
+        const float* bc = reinterpret_cast<const float*>(at(base / SS_TT));
+        const float2* step = sdt[(base / SS_TT) & 1] + ch;
+        float done[SS_TT / 4];                                // y of this lane's token of every four
+#pragma unroll
+        for (int g = 0; g < SS_TT; g += 4) {
             float part[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
-                const float dt = __shfl_sync(0xffffffffu, my_dt, k, 4), dx = __shfl_sync(0xffffffffu, my_dx, k, 4);
-                const float* row = &sBC[buf][g + k][0];
+                const float2 d = step[(g + k) * SS_CH];
+                if (MODE == SS_ADDS) dt_sum += d.x;
+                const float* row = bc + (g + k) * 2 * NP;
                 float y = 0.f;
 #pragma unroll
                 for (int i = 0; i < NPT; i += V) {
@@ -149,7 +228,7 @@ __global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(const ScanPa
                     if (MODE != SS_ADDS) ss_load<V>(row + NP + ss_state_of<V>(q, i), cv);
 #pragma unroll
                     for (int j = 0; j < V; ++j) {
-                        s[i + j] = fmaf(ss_exp2(dt * A2[i + j]), s[i + j], dx * b[j]);
+                        s[i + j] = fmaf(ss_exp2(d.x * A2[i + j]), s[i + j], d.y * b[j]);
                         if (MODE != SS_ADDS) y = fmaf(s[i + j], cv[j], y);
                     }
                 }
@@ -162,29 +241,29 @@ __global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(const ScanPa
                 const float s0 = up ? part[0] : part[2], s1 = up ? part[1] : part[3];
                 const float b0 = a0 + __shfl_xor_sync(0xffffffffu, s0, 2), b1 = a1 + __shfl_xor_sync(0xffffffffu, s1, 2);
                 const float mine = odd ? b1 : b0, other = odd ? b0 : b1;
-                const float y = fmaf(skip, my_x, mine + __shfl_xor_sync(0xffffffffu, other, 1));
-                if (in && live) og[(size_t)(t0 + base + g + q) * p.C] = vm_from_float<T>(y * silu_f(my_z));
+                done[g / 4] = mine + __shfl_xor_sync(0xffffffffu, other, 1);
             }
         }
-        __syncthreads();
+        if (MODE != SS_ADDS) {
+            const T* xs = reinterpret_cast<const T*>(bc + SS_TT * 2 * NP + SS_TT * SS_CH) + ch;
+            const T* zs = xs + SS_TT * SS_CH;
+#pragma unroll
+            for (int g = 0; g < SS_TT; g += 4) {
+                const float y = fmaf(skip, vm_to_float(xs[(g + q) * SS_CH]), done[g / 4]);
+                if (base + g + q < len && live) og[(size_t)(t0 + base + g + q) * p.C] = vm_from_float<T>(y * ss_silu(vm_to_float(zs[(g + q) * SS_CH])));
+            }
+        }
     }
-    if (MODE == SS_WHOLE && live) {
+    asm volatile("cp.async.wait_all;\n" ::);
+    float* keep = MODE == SS_WHOLE ? S : (MODE == SS_ADDS ? piece_S : nullptr);
+    if (keep && live) {
 #pragma unroll
         for (int i = 0; i < NPT; ++i) {
             const int n = ss_state_of<V>(q, i);
-            if (n < p.N) S[n] = s[i];
+            if (n < p.N) keep[n] = s[i];
         }
     }
-    if (MODE == SS_ADDS && live) {
-#pragma unroll
-        for (int i = 0; i < NPT; ++i) {
-            const int n = ss_state_of<V>(q, i);
-            if (n < p.N) piece_S[n] = s[i];
-        }
-        dt_sum += __shfl_xor_sync(0xffffffffu, dt_sum, 1, 4);
-        dt_sum += __shfl_xor_sync(0xffffffffu, dt_sum, 2, 4);
-        if (q == 0) p.dt_sums[(size_t)blockIdx.y * p.C + c] = dt_sum;
-    }
+    if (MODE == SS_ADDS && live && q == 0) p.dt_sums[(size_t)blockIdx.y * p.C + c] = dt_sum;
 }
 
 // grid (ceil(C N / 256), sequences): a thread carries one state value through its sequence's pieces
@@ -304,7 +383,14 @@ int launch_scan_mode(const ScanParams& p, int n_pieces, cudaStream_t stream) {
     const dim3 grid((p.C + SS_CH - 1) / SS_CH, n_pieces);
 #define VM_SEL(NPT)                                                                             \
     if (p.N <= 4 * NPT) {                                                                       \
-        selective_scan_kernel<T, NPT, MODE><<<grid, SS_THREADS, 0, stream>>>(p);                \
+        constexpr int smem = SS_STAGES * ss_stage_bytes<T, NPT>();                              \
+        static bool raised = false;                                                             \
+        if (smem > 32 * 1024 && !raised) {                                                      \
+            cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<T, NPT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
+            if (e != cudaSuccess) return (int)e;                                                \
+            raised = true;                                                                      \
+        }                                                                                       \
+        selective_scan_kernel<T, NPT, MODE><<<grid, SS_THREADS, smem, stream>>>(p);             \
         return vm_launch_status();                                                              \
     }
     VM_SEL(2) VM_SEL(4) VM_SEL(6) VM_SEL(8) VM_SEL(12) VM_SEL(16) VM_SEL(32)
@@ -360,6 +446,9 @@ VM_API int vm_selective_scan(const void* x, const float* dt, int ldt, const floa
     p.cu_tokens = cu_tokens; p.slots = slots; p.out = out;
     p.ldt = ldt; p.ldr = ldr; p.b_col = b_col; p.ldz = ldz; p.B = B; p.C = C; p.N = N;
     p.piece = scratch ? piece : 0x3fffffff;
+    const int e16 = act_dtype == VM_F32 ? 4 : 8;              // values of the activation dtype in 16 bytes
+    const uintptr_t bases = (uintptr_t)x | (uintptr_t)dt | (uintptr_t)r | (uintptr_t)z;
+    p.vec = bases % 16 == 0 && C % e16 == 0 && ldz % e16 == 0 && ldt % 4 == 0 && ldr % 4 == 0 && b_col % 4 == 0 && N % 4 == 0 ? 1 : 0;
     if (act_dtype == VM_F32) return launch_scan<float>(p, n_pieces, stream);
     if (act_dtype == VM_BF16) return launch_scan<__nv_bfloat16>(p, n_pieces, stream);
     return VM_ERR_UNSUPPORTED;

@@ -516,13 +516,14 @@ void attention(StepContext& ctx, const void* q, int q_row_stride, const KVView& 
 
 int selective_piece_tokens(const StepContext& ctx, int C) {
     if (ctx.T_cap < 64) return 0;
-    // a warp takes 8 channels; with about one warp for each of an SM's four schedulers one pass over the tokens is as fast as the pieces'
-    // two passes and their carry
-    const long long warps = static_cast<long long>(ctx.B_cap) * ((C + 7) / 8), want = 4ll * sm_count();
-    if (10 * warps >= 6 * want) return 0;
-    const long long pieces = (3 * want + warps - 1) / warps;      // per sequence of equal length: about three warps for each scheduler
+    // A warp takes 8 channels.  One pass over the tokens costs the latency of a warp's chain per token, however many warps there are; the pieces
+    // cost two passes and a carry (measured, 2,048 tokens: 4,096 channels 240 us whole, 153 us in pieces of 256; 1,024 channels 236 / 58 us in
+    // pieces of 128; four prompts of 2,048 tokens and 2,048 channels: 266 / 282 us).
+    const long long warps = static_cast<long long>(ctx.B_cap) * ((C + 7) / 8), sm_warps = 4ll * sm_count();
+    if (2 * warps >= 3 * sm_warps) return 0;
+    const long long pieces = (6 * sm_warps + warps - 1) / warps;      // of a sequence: about six warps for each of an SM's four schedulers
     const long long tokens = (ctx.T_cap / std::max(1, ctx.B_cap) + pieces - 1) / pieces;
-    return static_cast<int>(std::max<long long>(32, (tokens + 31) / 32 * 32));
+    return static_cast<int>(std::max<long long>(64, (tokens + 31) / 32 * 32));
 }
 
 void attention_biased(StepContext& ctx, const void* q, int q_row_stride, const KVView& kv, void* out, int H, int Hkv, int Dk, int Dv, float scale,
