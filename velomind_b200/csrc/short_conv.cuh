@@ -30,6 +30,58 @@ __global__ void conv_silu_kernel(const T* __restrict__ proj, int ld, int u_col, 
     out[(size_t)t * C + c] = vm_from_float<T>(silu_f(acc));
 }
 
+// Two neighbouring channels a thread (one load of both), CONV_TOK tokens one after another with the K - 1 earlier inputs carried in registers.
+// The same sum in the same order as above.
+constexpr int CONV_TOK = 8;
+__device__ __forceinline__ float2 conv_load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 conv_load2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void conv_store2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void conv_store2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+
+template <typename T, int K>
+__global__ void __launch_bounds__(128)
+conv_silu_pairs_kernel(const T* __restrict__ proj, int ld, int u_col, const float* __restrict__ taps, const float* __restrict__ bias,
+                       const float* __restrict__ state, int state_floats, int conv_off, const int* __restrict__ seq_of_token, const int* __restrict__ cu_tokens,
+                       const int* __restrict__ slots, int n_tokens, int C, T* __restrict__ out) {
+    const int c = 2 * (blockIdx.x * blockDim.x + threadIdx.x), t0 = blockIdx.y * CONV_TOK;
+    if (c >= C) return;
+    float2 w[K], u[K];                                     // taps; u[K - 1] the current token's input, u[K - 1 - b] that of b tokens ago
+#pragma unroll
+    for (int k = 0; k < K; ++k) w[k] = make_float2(taps[(size_t)c * K + k], taps[(size_t)(c + 1) * K + k]);
+    const float2 b2 = bias ? make_float2(bias[c], bias[c + 1]) : make_float2(0.f, 0.f);
+    const T* base = proj + u_col + c;
+    float2 fresh[CONV_TOK];                                // (all loads before the first use)
+#pragma unroll
+    for (int i = 0; i < CONV_TOK; ++i) fresh[i] = t0 + i < n_tokens ? conv_load2(base + (size_t)(t0 + i) * ld) : make_float2(0.f, 0.f);
+    int seq = -1;
+#pragma unroll
+    for (int i = 0; i < CONV_TOK; ++i) {
+        const int t = t0 + i;
+        if (t >= n_tokens) break;
+        const int sq = seq_of_token[t];
+        if (sq != seq) {                                   // the first token here, or another sequence's first one: the inputs before it
+            seq = sq;
+            const int local = t - cu_tokens[sq];
+            const float* kept = state + (size_t)slots[sq] * state_floats + conv_off;
+#pragma unroll
+            for (int back = 1; back < K; ++back) {
+                if (local - back >= 0) u[K - 1 - back] = conv_load2(base + (size_t)(t - back) * ld);
+                else u[K - 1 - back] = make_float2(kept[(size_t)(K - 1 + local - back) * C + c], kept[(size_t)(K - 1 + local - back) * C + c + 1]);
+            }
+        }
+        u[K - 1] = fresh[i];
+        float2 acc = b2;
+#pragma unroll
+        for (int k = 0; k < K; ++k) {
+            acc.x = fmaf(w[k].x, u[k].x, acc.x);
+            acc.y = fmaf(w[k].y, u[k].y, acc.y);
+        }
+        conv_store2(out + (size_t)t * C + c, make_float2(__fdividef(acc.x, 1.0f + __expf(-acc.x)), __fdividef(acc.y, 1.0f + __expf(-acc.y))));
+#pragma unroll
+        for (int k = 0; k + 1 < K; ++k) u[k] = u[k + 1];
+    }
+}
+
 // A block per sequence, a thread per channel: the last K - 1 inputs after this step (older ones move up, new ones come in).
 template <typename T>
 __global__ void conv_keep_kernel(const T* __restrict__ proj, int ld, int u_col, float* __restrict__ state, int state_floats, int conv_off,
@@ -81,8 +133,17 @@ int launch_short_conv(const void* proj, int ld, int u_col, const float* taps, co
                       conv_off, slots, B, C, K, (T*)out);
     } else {
         if (T_ > 65535) return VM_ERR_UNSUPPORTED;
-        conv_silu_kernel<T><<<dim3((C + 255) / 256, T_), 256, 0, stream>>>((const T*)proj, ld, u_col, taps, bias, state, state_floats, conv_off, positions,
-                                                                           seq_of_token, cu_tokens, slots, T_, C, K, (T*)out);
+        const bool pairs = C % 2 == 0 && ld % 2 == 0 && u_col % 2 == 0 && (((uintptr_t)proj | (uintptr_t)out) & (2 * sizeof(T) - 1)) == 0;
+#define VM_CONV(K_)                                                                                                                          \
+    if (pairs && K == K_)                                                                                                                    \
+        conv_silu_pairs_kernel<T, K_><<<dim3((C / 2 + 127) / 128, (T_ + CONV_TOK - 1) / CONV_TOK), 128, 0, stream>>>(                          \
+            (const T*)proj, ld, u_col, taps, bias, state, state_floats, conv_off, seq_of_token, cu_tokens, slots, T_, C, (T*)out);
+        VM_CONV(2)
+        else VM_CONV(3)
+        else VM_CONV(4)
+#undef VM_CONV
+        else conv_silu_kernel<T><<<dim3((C + 255) / 256, T_), 256, 0, stream>>>((const T*)proj, ld, u_col, taps, bias, state, state_floats, conv_off, positions,
+                                                                                seq_of_token, cu_tokens, slots, T_, C, K, (T*)out);
         if (K > 1)
             conv_keep_kernel<T><<<dim3(B, (C + 255) / 256), 256, 0, stream>>>((const T*)proj, ld, u_col, state, state_floats, conv_off, cu_tokens, slots, C, K);
     }
