@@ -532,11 +532,12 @@ VM_API int vm_expert_router_groups(const void* x, const float* norm_w, float eps
     if (top > (n_out / group_count) * group_keep) return VM_ERR_BAD_ARG;
     const size_t smem = (size_t)(hidden + 2 * n_out + group_count) * sizeof(float);
     if (smem > 48 * 1024) return VM_ERR_UNSUPPORTED;
+    const int threads = T <= 148 && n_out > 8 ? 1024 : 256;      // few tokens: a warp for each output or two (the block's latency is the step's)
     if (act_dtype == VM_F32)
-        vm_launch_pdl(router_scored_kernel<float>, dim3(T), dim3(256), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top, group_count,
+        vm_launch_pdl(router_scored_kernel<float>, dim3(T), dim3(threads), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top, group_count,
                       group_keep, group_top, scale, score_kind, normalize, chosen, weight);
     else if (act_dtype == VM_BF16)
-        vm_launch_pdl(router_scored_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top,
+        vm_launch_pdl(router_scored_kernel<__nv_bfloat16>, dim3(T), dim3(threads), smem, stream, x, norm_w, eps, w_router, correction, hidden, n_out, top,
                       group_count, group_keep, group_top, scale, score_kind, normalize, chosen, weight);
     else return VM_ERR_UNSUPPORTED;
     return vm_launch_status();

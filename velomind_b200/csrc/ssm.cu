@@ -10,6 +10,7 @@
 // What a sequence keeps (float32, in its slot's state area): S [H, N, P], then the last K - 1 convolution inputs [K - 1, C].
 // The state is zero when a slot is opened, which is also what "zeros before the start" asks of the convolution.
 // Step sizes, decays, the state and the sums over it are float32 whatever the activation dtype.
+#include "mma.cuh"
 #include "short_conv.cuh"
 
 namespace {
@@ -354,6 +355,256 @@ ssm_chunk_finish_kernel(const T* __restrict__ xbc, int C, const float* __restric
     }
 }
 
+// ------------------------------------------------------------------------------------------------ the same on the tensor cores (bfloat16)
+// The convolved inputs are bfloat16 already, so C B^T, B^T (w x), P x and C S have one factor that bfloat16 holds exactly; the other one (step
+// sizes and decays in it, or the state) is float32 and enters as the sum of three bfloat16 numbers, which keep all its 24 bits; sums are float32.
+// Pass 1: what a chunk adds to the state.  Pass 2 as above.  Pass 3: scores, decays and mask on them, their product with x, the old state's share
+// and the skip term in one kernel; y is written once.  Four warps a block; in pass 3 a warp owns 16 of the chunk's tokens, in pass 1 rows of
+// 16 state values.  States and values per head in multiples of 16.
+constexpr int MMA_THREADS = 128;
+
+// a pair of float32 as three pairs of bfloat16 whose sums they are
+__device__ __forceinline__ void split3(float a, float b, unsigned (&u)[3]) {
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+        u[k] = *reinterpret_cast<const unsigned*>(&h);
+        a -= __low2float(h);
+        b -= __high2float(h);
+    }
+}
+
+// step sizes and running sums of the log decays of a chunk's tokens, by the first warp (a token and the next one per lane)
+template <typename T>
+__device__ __forceinline__ void chunk_steps(const T* __restrict__ proj, int ld, int dt_col, int h, float bias, float rate, int t0, int len, float* sdt, float* scum) {
+    const int lane = threadIdx.x;
+    float d[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int t = 2 * lane + k;
+        d[k] = t < len ? softplus_f(vm_to_float(proj[(size_t)(t0 + t) * ld + dt_col + h]) + bias) : 0.f;
+        sdt[t] = d[k];
+    }
+    const float pair = rate * d[0] + rate * d[1];
+    float sum = pair;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += v;
+    }
+    scum[2 * lane + 1] = sum;
+    scum[2 * lane] = sum - rate * d[1];
+}
+
+// rows of a chunk (zeros past its end) into shared memory, 16 bytes at a time: columns [col, col + n) of xbc into rows of `pitch`, zeros up to n_pad
+__device__ __forceinline__ void chunk_rows(const __nv_bfloat16* __restrict__ xbc, int C, int col, int n, int n_pad, int t0, int len, __nv_bfloat16* dst, int pitch) {
+    const int ch = n_pad / 8;
+    for (int i = threadIdx.x; i < CL * ch; i += MMA_THREADS) {
+        const int t = i / ch, c = 8 * (i - t * ch);
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (t < len && c < n) v = *reinterpret_cast<const uint4*>(xbc + (size_t)(t0 + t) * C + col + c);
+        *reinterpret_cast<uint4*>(dst + t * pitch + c) = v;
+    }
+}
+
+template <int PB>      // values per head, in units of 16 columns (padded with zeros)
+__global__ void __launch_bounds__(MMA_THREADS)
+ssm_mma_adds_kernel(const __nv_bfloat16* __restrict__ xbc, int C, const __nv_bfloat16* __restrict__ proj, int ld, int dt_col, const float* __restrict__ dt_bias,
+                    const float* __restrict__ A_log, const int* __restrict__ cu_tokens, int B, float* __restrict__ dS, float* __restrict__ decay_out,
+                    int H, int P, int N, int G) {
+    constexpr int XP = PB * 16 + 8;
+    extern __shared__ __align__(16) unsigned char raw[];
+    __shared__ float sdt[CL], scum[CL];
+    __nv_bfloat16* sX = reinterpret_cast<__nv_bfloat16*>(raw);      // [3][CL][XP]: w x in three parts
+    __nv_bfloat16* sB = sX + 3 * CL * XP;                           // [CL][N + 8]
+    const int NP = N + 8;
+    int seq, t0, len;
+    if (!chunk_where(cu_tokens, B, blockIdx.x, seq, t0, len)) return;
+    const int h = blockIdx.y, g = h / (H / G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int inner = H * P;
+    chunk_rows(xbc, C, inner + g * N, N, N, t0, len, sB, NP);
+    if (warp == 0) chunk_steps(proj, ld, dt_col, h, dt_bias ? dt_bias[h] : 0.f, -expf(A_log[h]), t0, len, sdt, scum);
+    __syncthreads();
+    const float c_last = scum[CL - 1];
+    for (int i = tid; i < CL * PB * 8; i += MMA_THREADS) {
+        const int s = i / (PB * 8), p = 2 * (i - s * PB * 8);
+        float2 x = make_float2(0.f, 0.f);
+        if (s < len && p < P) x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(xbc + (size_t)(t0 + s) * C + h * P + p));
+        const float w = sdt[s] * __expf(c_last - scum[s]);
+        unsigned u[3];
+        split3(w * x.x, w * x.y, u);
+#pragma unroll
+        for (int k = 0; k < 3; ++k) *reinterpret_cast<unsigned*>(sX + (k * CL + s) * XP + p) = u[k];
+    }
+    if (tid == 0) decay_out[(size_t)blockIdx.x * H + h] = expf(c_last);
+    __syncthreads();
+    float* out = dS + ((size_t)blockIdx.x * H + h) * N * P;
+    for (int mt = warp; mt < N / 16; mt += MMA_THREADS / 32) {
+        float acc[PB * 2][4];
+#pragma unroll
+        for (int i = 0; i < PB * 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < CL / 16; ++kk) {
+            unsigned a0, a1, a2, a3;      // (state value, token) from rows of (token, state value)
+            vm_ldmatrix_x4_trans(a0, a1, a2, a3, sB + (kk * 16 + (lane & 7) + 8 * (lane >> 4)) * NP + mt * 16 + 8 * ((lane >> 3) & 1));
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+#pragma unroll
+                for (int nb = 0; nb < PB * 2; nb += 2) {
+                    unsigned b0, b1, b2, b3;
+                    vm_ldmatrix_x4_trans(b0, b1, b2, b3, sX + (k * CL + kk * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * XP + nb * 8 + 8 * (lane >> 4));
+                    vm_mma_bf16_16816(acc[nb], a0, a1, a2, a3, b0, b1);
+                    vm_mma_bf16_16816(acc[nb + 1], a0, a1, a2, a3, b2, b3);
+                }
+        }
+        const int n = mt * 16 + (lane >> 2);
+#pragma unroll
+        for (int nb = 0; nb < PB * 2; ++nb) {
+            const int p = nb * 8 + 2 * (lane & 3);
+            if (p >= P) continue;
+            *reinterpret_cast<float2*>(out + (size_t)n * P + p) = make_float2(acc[nb][0], acc[nb][1]);
+            *reinterpret_cast<float2*>(out + (size_t)(n + 8) * P + p) = make_float2(acc[nb][2], acc[nb][3]);
+        }
+    }
+}
+
+template <int PB>
+__global__ void __launch_bounds__(MMA_THREADS)
+ssm_mma_out_kernel(const __nv_bfloat16* __restrict__ xbc, int C, const __nv_bfloat16* __restrict__ proj, int ld, int dt_col, const float* __restrict__ dt_bias,
+                   const float* __restrict__ A_log, const float* __restrict__ Dskip, const int* __restrict__ cu_tokens, int B, float* __restrict__ y,
+                   const float* __restrict__ S_start, int H, int P, int N, int G) {
+    constexpr int XP = PB * 16 + 8;
+    extern __shared__ __align__(16) unsigned char raw[];
+    __shared__ float sdt[CL], scum[CL];
+    const int NP = N + 8;
+    __nv_bfloat16* sX = reinterpret_cast<__nv_bfloat16*>(raw);      // [CL][XP]
+    __nv_bfloat16* sS = sX + CL * XP;                               // [3][NT][XP]: 64 rows of the state in three parts
+    __nv_bfloat16* sC = sS + 3 * NT * XP;                           // [CL][NP]
+    __nv_bfloat16* sB = sC + CL * NP;                               // [CL][NP]
+    int seq, t0, len;
+    if (!chunk_where(cu_tokens, B, blockIdx.x, seq, t0, len)) return;
+    const int h = blockIdx.y, g = h / (H / G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int inner = H * P;
+    chunk_rows(xbc, C, inner + g * N, N, N, t0, len, sB, NP);
+    chunk_rows(xbc, C, inner + G * N + g * N, N, N, t0, len, sC, NP);
+    chunk_rows(xbc, C, h * P, P, PB * 16, t0, len, sX, XP);
+    if (warp == 0) chunk_steps(proj, ld, dt_col, h, dt_bias ? dt_bias[h] : 0.f, -expf(A_log[h]), t0, len, sdt, scum);
+    const float* S = S_start + ((size_t)blockIdx.x * H + h) * N * P;
+    float o[PB * 2][4];
+#pragma unroll
+    for (int i = 0; i < PB * 2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    const __nv_bfloat16* c_rows = sC + (warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * NP + 8 * (lane >> 4);
+    // ---- the old state's share: o = C S
+    for (int n0 = 0; n0 < N; n0 += NT) {
+        const int rows = min(NT, N - n0);
+        __syncthreads();                                            // (the rows above are there; the tile before is read)
+        for (int i = tid; i < rows * PB * 8; i += MMA_THREADS) {
+            const int n = i / (PB * 8), p = 2 * (i - n * PB * 8);
+            const float2 v = p < P ? *reinterpret_cast<const float2*>(S + (size_t)(n0 + n) * P + p) : make_float2(0.f, 0.f);
+            unsigned u[3];
+            split3(v.x, v.y, u);
+#pragma unroll
+            for (int k = 0; k < 3; ++k) *reinterpret_cast<unsigned*>(sS + (k * NT + n) * XP + p) = u[k];
+        }
+        __syncthreads();
+        for (int kk = 0; kk < rows / 16; ++kk) {
+            unsigned a0, a1, a2, a3;
+            vm_ldmatrix_x4(a0, a1, a2, a3, c_rows + n0 + kk * 16);
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+#pragma unroll
+                for (int nb = 0; nb < PB * 2; nb += 2) {
+                    unsigned b0, b1, b2, b3;
+                    vm_ldmatrix_x4_trans(b0, b1, b2, b3, sS + (k * NT + kk * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * XP + nb * 8 + 8 * (lane >> 4));
+                    vm_mma_bf16_16816(o[nb], a0, a1, a2, a3, b0, b1);
+                    vm_mma_bf16_16816(o[nb + 1], a0, a1, a2, a3, b2, b3);
+                }
+        }
+    }
+    // ---- scores of this warp's 16 tokens with the chunk's tokens up to them
+    float sc[CL / 8][4];
+#pragma unroll
+    for (int i = 0; i < CL / 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+    for (int kk = 0; kk < N / 16; ++kk) {
+        unsigned a0, a1, a2, a3;
+        vm_ldmatrix_x4(a0, a1, a2, a3, c_rows + kk * 16);
+#pragma unroll
+        for (int nb = 0; nb < CL / 8; nb += 2) {
+            if (nb > 2 * warp) continue;                            // (tokens after all of this warp's)
+            unsigned b0, b1, b2, b3;
+            vm_ldmatrix_x4(b0, b1, b2, b3, sB + (nb * 8 + (lane & 7) + 8 * (lane >> 4)) * NP + kk * 16 + 8 * ((lane >> 3) & 1));
+            vm_mma_bf16_16816(sc[nb], a0, a1, a2, a3, b0, b1);
+            vm_mma_bf16_16816(sc[nb + 1], a0, a1, a2, a3, b2, b3);
+        }
+    }
+    const int ta = warp * 16 + (lane >> 2), tb = ta + 8, t4 = lane & 3;
+    const float ca = scum[ta], cb = scum[tb], ea = __expf(ca), eb = __expf(cb);
+#pragma unroll
+    for (int i = 0; i < PB * 2; ++i) { o[i][0] *= ea; o[i][1] *= ea; o[i][2] *= eb; o[i][3] *= eb; }
+    // ---- decays, step sizes and mask on the scores; their product with x
+#pragma unroll
+    for (int kk = 0; kk < CL / 16; ++kk) {
+        if (kk > warp) continue;
+        unsigned pa[4][3];                                          // the A fragment of 16 x 16 scores, in three parts
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int s = kk * 16 + half * 8 + 2 * t4;
+            const float* v = sc[kk * 2 + half];
+            const float d0 = sdt[s], d1 = sdt[s + 1], c0 = scum[s], c1 = scum[s + 1];
+            split3(s <= ta ? v[0] * __expf(ca - c0) * d0 : 0.f, s + 1 <= ta ? v[1] * __expf(ca - c1) * d1 : 0.f, pa[half * 2]);
+            split3(s <= tb ? v[2] * __expf(cb - c0) * d0 : 0.f, s + 1 <= tb ? v[3] * __expf(cb - c1) * d1 : 0.f, pa[half * 2 + 1]);
+        }
+#pragma unroll
+        for (int nb = 0; nb < PB * 2; nb += 2) {
+            unsigned b0, b1, b2, b3;
+            vm_ldmatrix_x4_trans(b0, b1, b2, b3, sX + (kk * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * XP + nb * 8 + 8 * (lane >> 4));
+#pragma unroll
+            for (int k = 0; k < 3; ++k) {
+                vm_mma_bf16_16816(o[nb], pa[0][k], pa[1][k], pa[2][k], pa[3][k], b0, b1);
+                vm_mma_bf16_16816(o[nb + 1], pa[0][k], pa[1][k], pa[2][k], pa[3][k], b2, b3);
+            }
+        }
+    }
+    const float skip = Dskip ? Dskip[h] : 0.f;
+#pragma unroll
+    for (int nb = 0; nb < PB * 2; ++nb) {
+        const int p = nb * 8 + 2 * t4;
+        if (p >= P) continue;
+        const float2 xa = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + ta * XP + p));
+        const float2 xb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + tb * XP + p));
+        if (ta < len) *reinterpret_cast<float2*>(y + (size_t)(t0 + ta) * inner + h * P + p) = make_float2(fmaf(skip, xa.x, o[nb][0]), fmaf(skip, xa.y, o[nb][1]));
+        if (tb < len) *reinterpret_cast<float2*>(y + (size_t)(t0 + tb) * inner + h * P + p) = make_float2(fmaf(skip, xb.x, o[nb][2]), fmaf(skip, xb.y, o[nb][3]));
+    }
+}
+
+// sizes the tensor-core passes take
+bool mma_fits(int C, int P, int N) { return P % 16 == 0 && P <= 128 && N % 16 == 0 && N <= 256 && C % 8 == 0; }
+
+template <int PB>
+int launch_chunks_mma(const __nv_bfloat16* xbc, int C, const __nv_bfloat16* proj, int ld, int dt_col, const float* dt_bias, const float* A_log, const float* Dskip,
+                      float* state, int state_floats, const int* cu_tokens, const int* slots, float* y, float* scratch, int B, int n_chunks, int H, int P, int N, int G,
+                      cudaStream_t stream) {
+    constexpr int XP = PB * 16 + 8;
+    float* dS = scratch;
+    float* decay = dS + (size_t)n_chunks * H * N * P;
+    const size_t smem1 = ((size_t)3 * CL * XP + (size_t)CL * (N + 8)) * 2, smem3 = ((size_t)CL * XP + (size_t)3 * NT * XP + (size_t)2 * CL * (N + 8)) * 2;
+    static bool raised = false;           // per instantiation, for the largest sizes it takes
+    if (!raised) {
+        const int most1 = (3 * CL * XP + CL * 264) * 2, most3 = (CL * XP + 3 * NT * XP + 2 * CL * 264) * 2;
+        if (cudaFuncSetAttribute(ssm_mma_adds_kernel<PB>, cudaFuncAttributeMaxDynamicSharedMemorySize, most1) != cudaSuccess) return vm_launch_status();
+        if (cudaFuncSetAttribute(ssm_mma_out_kernel<PB>, cudaFuncAttributeMaxDynamicSharedMemorySize, most3) != cudaSuccess) return vm_launch_status();
+        raised = true;
+    }
+    ssm_mma_adds_kernel<PB><<<dim3(n_chunks, H), MMA_THREADS, smem1, stream>>>(xbc, C, proj, ld, dt_col, dt_bias, A_log, cu_tokens, B, dS, decay, H, P, N, G);
+    int st = vm_launch_status();
+    if (st) return st;
+    ssm_chunk_carry_kernel<<<dim3(B * H, (N * P + 255) / 256), 256, 0, stream>>>(dS, decay, state, state_floats, cu_tokens, slots, B, H, P, N);
+    st = vm_launch_status();
+    if (st) return st;
+    ssm_mma_out_kernel<PB><<<dim3(n_chunks, H), MMA_THREADS, smem3, stream>>>(xbc, C, proj, ld, dt_col, dt_bias, A_log, Dskip, cu_tokens, B, y, dS, H, P, N, G);
+    return vm_launch_status();
+}
+
 template <typename T, int PC>
 int launch_chunks_pc(const void* xbc, int C, const void* proj, int ld, int dt_col, const float* dt_bias, const float* A_log, const float* Dskip,
                      float* state, int state_floats, const int* cu_tokens, const int* slots, float* y, float* scratch, int T_, int B, int n_chunks,
@@ -385,6 +636,17 @@ template <typename T>
 int launch_chunks(const void* xbc, int C, const void* proj, int ld, int dt_col, const float* dt_bias, const float* A_log, const float* Dskip, float* state,
                   int state_floats, const int* cu_tokens, const int* slots, float* y, float* scratch, int T_, int B, int n_chunks, int H, int P, int N,
                   int G, cudaStream_t stream) {
+    if constexpr (sizeof(T) == 2) {
+        if (mma_fits(C, P, N) && ((uintptr_t)xbc & 15) == 0) {
+#define VM_CHM(PB)                                                                                                                                       \
+    return launch_chunks_mma<PB>((const T*)xbc, C, (const T*)proj, ld, dt_col, dt_bias, A_log, Dskip, state, state_floats, cu_tokens, slots, y, scratch, B, \
+                                 n_chunks, H, P, N, G, stream)
+            if (P <= 32) VM_CHM(2);
+            if (P <= 64) VM_CHM(4);
+            VM_CHM(8);
+#undef VM_CHM
+        }
+    }
 #define VM_CH(PC)                                                                                                                                  \
     return launch_chunks_pc<T, PC>(xbc, C, proj, ld, dt_col, dt_bias, A_log, Dskip, state, state_floats, cu_tokens, slots, y, scratch, T_, B, n_chunks, H, \
                                    P, N, G, stream)
@@ -417,6 +679,51 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, const T* __
             const int c = part * per + i;
             out[(size_t)t * inner + c] = vm_from_float<T>(gs[c] * inv * w[c]);
         }
+    }
+}
+
+// One part, rows of 4 n values: a thread keeps RUNS runs of four values in registers (inner <= 4 RUNS blockDim)
+__device__ __forceinline__ float4 gn_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 gn_load4(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void gn_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void gn_store4(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(vm_pack_bf16(v.x, v.y), vm_pack_bf16(v.z, v.w));
+}
+
+template <typename T, int RUNS>
+__global__ void gated_norm_vec_kernel(const float* __restrict__ y, const T* __restrict__ proj, int ld, int z_col, const float* __restrict__ w, float eps, int inner,
+                                      T* __restrict__ out) {
+    __shared__ float red[32];
+    vm_pdl_launch_dependents();
+    float4 wv[RUNS], v[RUNS];
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {                       // (constants: they may be read before the wait)
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        wv[c] = i < inner ? gn_load4(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    vm_pdl_wait();
+    const size_t t = blockIdx.x;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i >= inner) continue;
+        const float4 z = gn_load4(proj + t * ld + z_col + i);
+        v[c] = gn_load4(y + t * inner + i);
+        v[c].x *= silu_f(z.x); v[c].y *= silu_f(z.y); v[c].z *= silu_f(z.z); v[c].w *= silu_f(z.w);
+        ss += v[c].x * v[c].x + v[c].y * v[c].y + v[c].z * v[c].z + v[c].w * v[c].w;
+    }
+    ss = vm_block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)inner + eps);
+#pragma unroll
+    for (int c = 0; c < RUNS; ++c) {
+        const int i = (threadIdx.x + c * blockDim.x) * 4;
+        if (i < inner) gn_store4(out + t * inner + i, make_float4(v[c].x * inv * wv[c].x, v[c].y * inv * wv[c].y, v[c].z * inv * wv[c].z, v[c].w * inv * wv[c].w));
     }
 }
 
@@ -463,6 +770,21 @@ int launch_mixer(const void* proj, int ld, const float* taps, const float* conv_
     else
         st = launch_scan<T>(xbc, C, proj, ld, dt_col, dt_bias, A_log, Dskip, state, state_floats, cu_tokens, slots, y, B, H, P, N, G, vm_sm_count(), stream);
     if (st) return st;
+    const uintptr_t at = (uintptr_t)y | (uintptr_t)proj | (uintptr_t)norm_w | (uintptr_t)out;
+    if (parts == 1 && inner % 4 == 0 && ld % 4 == 0 && at % 16 == 0 && inner <= 16384) {
+        // few rows: as many threads as there are runs of four (the row's latency); many: two to eight runs a thread
+        int threads = T_ > 148 ? 256 : 1024;
+        while (threads > 128 && threads * 4 > 2 * inner) threads /= 2;
+        while (threads < 1024 && threads * 32 < inner) threads *= 2;
+        const int runs = (inner / 4 + threads - 1) / threads;
+#define VM_GN(R_) vm_launch_pdl(gated_norm_vec_kernel<T, R_>, dim3(T_), dim3(threads), 0, stream, (const float*)y, (const T*)proj, ld, 0, norm_w, eps, inner, (T*)out)
+        if (runs <= 1) VM_GN(1);
+        else if (runs <= 2) VM_GN(2);
+        else if (runs <= 4) VM_GN(4);
+        else VM_GN(8);
+#undef VM_GN
+        return vm_launch_status();
+    }
     vm_launch_pdl(gated_group_norm_kernel<T>, dim3(T_), dim3(256), (size_t)inner * sizeof(float), stream, (const float*)y, (const T*)proj, ld, 0, norm_w, eps,
                   inner, parts, (T*)out);
     return vm_launch_status();
