@@ -469,6 +469,23 @@ int launch_scaled_sum(float* h, const T* a, float ca, const T* a2, float ca2, co
 // ------------------------------------------------------------------------------------------------ a token's own row, gated
 // out[t, i] = gelu_tanh(z[t, i]) * table[token_t, off + i]; z float32 [T, ldz], table rows of ld_table values in W.  A token outside the
 // table reads its first row (the embedding, which reads the same token, reports it).
+__device__ __forceinline__ float gtr_gelu(float v) {      // 0.5 v (1 + tanh(u)) = v sigmoid(2 u)
+    return v / (1.0f + expf(-1.5957691216057308f * (v + 0.044715f * v * v * v)));
+}
+
+// four neighbouring columns a thread
+template <typename W, typename T>
+__global__ void gated_token_rows_vec_kernel(const float* __restrict__ z, int ldz, const int* __restrict__ tokens, const W* __restrict__ table, long long ld_table,
+                                            int off, int vocab, T* __restrict__ out, int n, int total4) {
+    vm_pdl_launch_dependents();
+    vm_pdl_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total4) return;
+    const int t = i / (n / 4), c = 4 * (i - t * (n / 4)), id = tokens[t];
+    const float4 v = ns_load4(z + (size_t)t * ldz + c), e = ns_load4(table + (size_t)(id >= 0 && id < vocab ? id : 0) * ld_table + off + c);
+    ns_store4(out + (size_t)t * n + c, make_float4(gtr_gelu(v.x) * e.x, gtr_gelu(v.y) * e.y, gtr_gelu(v.z) * e.z, gtr_gelu(v.w) * e.w));
+}
+
 template <typename W, typename T>
 __global__ void gated_token_rows_kernel(const float* __restrict__ z, int ldz, const int* __restrict__ tokens, const W* __restrict__ table, long long ld_table,
                                         int off, int vocab, T* __restrict__ out, int n, long long total) {
@@ -478,7 +495,7 @@ __global__ void gated_token_rows_kernel(const float* __restrict__ z, int ldz, co
         const long long t = i / n;
         const int c = (int)(i - t * n), id = tokens[t];
         const float v = z[t * ldz + c], e = vm_to_float(table[(size_t)(id >= 0 && id < vocab ? id : 0) * ld_table + off + c]);
-        out[i] = vm_from_float<T>(0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))) * e);
+        out[i] = vm_from_float<T>(gtr_gelu(v) * e);
     }
 }
 
@@ -724,11 +741,16 @@ VM_API int vm_gated_token_rows(const float* z, int ldz, const int* tokens, const
     if (n <= 0 || ldz < n || off < 0 || ld_table < off + n || vocab <= 0) return VM_ERR_BAD_ARG;
     const long long total = (long long)T * n, want = (total + 255) / 256;
     const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
+    const uintptr_t at = (uintptr_t)z | (uintptr_t)table | (uintptr_t)out;
+    const bool vec = n % 4 == 0 && ldz % 4 == 0 && ld_table % 4 == 0 && off % 4 == 0 && at % 16 == 0 && total < (1ll << 31);
+    const int total4 = (int)(total / 4);
 #define VM_GTR(W, T_) \
-    vm_launch_pdl(gated_token_rows_kernel<W, T_>, grid, dim3(256), 0, stream, z, ldz, tokens, (const W*)table, ld_table, off, vocab, (T_*)out, n, total)
-    if (table_dtype == VM_F32 && act_dtype == VM_F32) VM_GTR(float, float);
-    else if (table_dtype == VM_F32 && act_dtype == VM_BF16) VM_GTR(float, __nv_bfloat16);
-    else if (table_dtype == VM_BF16 && act_dtype == VM_BF16) VM_GTR(__nv_bfloat16, __nv_bfloat16);
+    if (vec) vm_launch_pdl(gated_token_rows_vec_kernel<W, T_>, dim3((total4 + 127) / 128), dim3(128), 0, stream, z, ldz, tokens, (const W*)table, ld_table, off, \
+                           vocab, (T_*)out, n, total4); \
+    else vm_launch_pdl(gated_token_rows_kernel<W, T_>, grid, dim3(256), 0, stream, z, ldz, tokens, (const W*)table, ld_table, off, vocab, (T_*)out, n, total)
+    if (table_dtype == VM_F32 && act_dtype == VM_F32) { VM_GTR(float, float); }
+    else if (table_dtype == VM_F32 && act_dtype == VM_BF16) { VM_GTR(float, __nv_bfloat16); }
+    else if (table_dtype == VM_BF16 && act_dtype == VM_BF16) { VM_GTR(__nv_bfloat16, __nv_bfloat16); }
     else return VM_ERR_UNSUPPORTED;
 #undef VM_GTR
     return vm_launch_status();
