@@ -165,6 +165,34 @@ TEST(groups_with_different_needs_have_their_own_storage) {
     no_keys.check();
 }
 
+TEST(a_chunk_group_gives_its_pages_back_when_the_chunk_is_over) {
+    CacheNeed chunk;
+    chunk.kind = CacheNeed::Chunk;
+    chunk.kv_heads = 1;
+    chunk.key_dim = chunk.value_dim = 16;
+    chunk.chunk = 100;
+    CacheNeed other = chunk;
+    other.chunk = 150;
+    CacheBook c({chunk, other, chunk}, {-1, -1, -1}, 64 * 16, 1024);
+    CHECK(c.groups.size() == 2 && c.where(2) == std::make_pair(0, 1));          // unlike chunks are unlike groups
+    const int s = c.open();
+    for (int n : {90, 100, 191, 192, 199, 200, 299, 300}) {
+        c.reserve(s, n);
+        c.commit(s, n);
+        // the next query, at place n, sees keys from its chunk's start on: the pages before that start's page are gone
+        for (int g = 0; g < 2; ++g) {
+            const int size = g == 0 ? 100 : 150, first = n - n % size, gone = std::min(first / VM_PAGE_TOKENS, (n + VM_PAGE_TOKENS - 1) / VM_PAGE_TOKENS);
+            CHECK(c.groups[g].blocks_begin[s] == gone);
+            CHECK(c.groups[g].pages.held_count() == (n + VM_PAGE_TOKENS - 1) / VM_PAGE_TOKENS - gone);
+        }
+        c.check();
+    }
+    c.close(s);
+    c.check();
+    chunk.chunk = 0;
+    THROWS(CacheError, "chunk > 0", CacheBook({chunk}, {-1}, 64 * 4, 256));
+}
+
 TEST(a_window_group_keeps_the_pages_of_its_first_tokens) {
     CacheNeed win;
     win.kind = CacheNeed::Window;

@@ -63,7 +63,7 @@ PARTS = {"attention": ("general_attention", attention_args, P.attention_mixer), 
          "mamba2": ("mamba2", mamba2_args, lambda h, w, m: P.mamba2_mixer(h, w, m, EPS)), "parallel": ("side_by_side", parallel_args, P.parallel_mixer),
          "dense": ("gated", dense_args, lambda h, w, m: P.clamped_unit(h, w, m["limit"])), "moe": ("routed_experts", moe_args, P.routed)}
 
-SLOWED = (4.0, 1.0, 4.0, 80)
+SLOWED = (5.0, 1.0, 3.0, 80)
 
 # name -> (kind, hidden, the configuration's own object)
 MECHANISMS = {
@@ -72,7 +72,7 @@ MECHANISMS = {
     # sizes the tensor-core kernel of prompts takes (bfloat16), a chunk of exactly one page, chunks that straddle pages and tiles
     "attention_tiles": ("attention", 128, C.attention(6, 2, 64, 32, 0.1, 64, 1000.0, 32)),
     "attention_tiles_over_pages": ("attention", 64, C.attention(2, 2, 32, 64, 0.3, 100, 500.0, None, SLOWED)),
-    "attention_tiles_wide": ("attention", 64, C.attention(2, 1, 128, 128, 0.1, 33, 20000.0, 64)),
+    "attention_tiles_wide": ("attention", 64, C.attention(2, 1, 128, 128, 0.1, 33, 7000.0, 96)),
     "attention_one_token": ("attention", 48, C.attention(2, 1, 8, 8, 0.4, 1)),
     "attention_small_chunk": ("attention", 48, C.attention(2, 2, 16, 16, 0.5, 7)),
     "attention_no_mask": ("attention", 64, C.attention(4, 4, 16, 24, 0.3, None, 100.0, 8)),
@@ -83,7 +83,7 @@ MECHANISMS = {
     "scan_many_taps": ("scan", 64, C.scan(40, 8, 12, 5)),
     "scan_state_one": ("scan", 48, C.scan(20, 1, 1, 2)),
     "scan_16": ("scan", 64, C.scan(128, 32, 16, 4)),
-    "scan_24": ("scan", 64, C.scan(72, 12, 24, 4)),
+    "scan_24": ("scan", 64, C.scan(72, 10, 24, 3)),
     "scan_40": ("scan", 48, C.scan(24, 16, 40, 4)),
     "scan_100": ("scan", 48, C.scan(32, 20, 100, 2)),
     "scan_128": ("scan", 64, C.scan(16, 8, 128, 4)),
